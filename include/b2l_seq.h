@@ -28,8 +28,9 @@ extern "C" {
 int b2l_seq_version(void);
 const char* b2l_seq_last_error(void);
 
-/* x[t, :] = table[token[t], :] * scale (f32 residual stream).  Tokens outside the table read row 0. */
-int b2l_seq_embed(const void* tokens, int tokens_i64, const void* table, int act_dtype, float scale, float* x,
+/* x[t, :] = table[token[t], :] * scale (f32 residual stream).  Tokens outside the table read row 0.  h (act [T, D], may be
+ * null) receives the same in the activation type, for layers that read the stream without a norm. */
+int b2l_seq_embed(const void* tokens, int tokens_i64, const void* table, int act_dtype, float scale, float* x, void* h,
                   int T, int D, int vocab, b2l_stream_t stream);
 
 /* out[t, :] = x / sqrt(mean(x^2) + eps) * w, x f32 -> out act.  `rows` (device int32[n_rows], may be null) picks
@@ -37,19 +38,20 @@ int b2l_seq_embed(const void* tokens, int tokens_i64, const void* table, int act
 int b2l_seq_rmsnorm(const float* x, const void* w, float eps, void* out, const int* rows, int n_rows, int D,
                     int act_dtype, b2l_stream_t stream);
 
-/* Post-norm residual step fused with the next pre-norm:
- *   x[t] += y[t] / sqrt(mean(y[t]^2) + eps) * w_post;   if w_next: h[t] = x[t] / sqrt(mean(x[t]^2) + eps) * w_next */
-int b2l_seq_norm_add_norm(const void* y, const void* w_post, float eps, float* x, const void* w_next, void* h, int T,
+/* Post-norm residual step fused with what the next sublayer reads:
+ *   x[t] += mult * y[t] / sqrt(mean(y[t]^2) + eps) * w_post;
+ *   h given: h[t] = x[t] / sqrt(mean(x[t]^2) + eps) * w_next, or, with w_next null, x[t] itself in the activation type */
+int b2l_seq_norm_add_norm(const void* y, const void* w_post, float eps, float mult, float* x, const void* w_next, void* h, int T,
                           int D, int act_dtype, b2l_stream_t stream);
 
 /* out[t, j] = act(gu[t, j]) * gu[t, F + j]  (gated feed-forward, both halves from one product).
  * B2L_SEQ_ACT_CLAMPED_SWISH is a gated unit with clamped halves: g = min(gu[t, j], limit),
  * u = clamp(gu[t, F + j], -limit, limit), out = g * sigmoid(1.702 g) * (u + 1).  `limit` is read by it alone. */
 enum { B2L_SEQ_ACT_GELU_TANH = 0, B2L_SEQ_ACT_SILU = 1, B2L_SEQ_ACT_SIGMOID = 2, B2L_SEQ_ACT_CLAMPED_SWISH = 3, B2L_SEQ_ACT_XIELU = 4,
-       B2L_SEQ_ACT_NONE = 5 };
+       B2L_SEQ_ACT_NONE = 5, B2L_SEQ_ACT_RELU2 = 6 };
 int b2l_seq_gated_act(const void* gu, int ldgu, void* out, int T, int F, int act, float limit, int act_dtype, b2l_stream_t stream);
 
-/* out[t, j] = act(in[t, j]) for an ungated feed-forward: gelu_tanh, silu, sigmoid, or B2L_SEQ_ACT_XIELU with its two
+/* out[t, j] = act(in[t, j]) for an ungated feed-forward: gelu_tanh, silu, sigmoid, relu2 (max(z, 0)^2), or B2L_SEQ_ACT_XIELU with its two
  * coefficients coef = {a, b} (f32, on the device; from the learned numbers p, q: a = softplus(p), b = 1/2 + softplus(q)):
  *   z > 0: a z^2 + z / 2;   z <= 0: b (exp(z) - 1 - z) + z / 2.
  * `coef` is read by xIELU alone.  out may be in (in place). */
@@ -119,6 +121,10 @@ typedef struct {
    * work_state: f32 [n_chunks][heads][V][K]; work_decay: f32 [n_chunks][heads][K] (per-channel decay) or
    * [n_chunks][heads].  b2l_seq_scan_chunks() says how many chunks a portion of T tokens wants (1 = sequential). */
   float* work_state; float* work_decay; int n_chunks;
+  /* A normaliser beside the matrix state (ones != 0; no skip, no delta rule): one more state column per head whose value
+   * is 1 at every step (times vscale), n <- d n + vscale k, kept in state_ones ([n_slots][heads][K] f32); out_ones
+   * (f32 [T, heads]) receives q_mult * n . q.  work_state then has V + 1 columns per head. */
+  int ones; float* state_ones; float* out_ones;
 } b2l_seq_scan_args;
 int b2l_seq_scan_chunks(int T, int delta);
 int b2l_seq_scan(const b2l_seq_scan_args* a, b2l_stream_t stream);
@@ -351,7 +357,7 @@ int b2l_seq_scale(float* z, size_t n, float mult, b2l_stream_t stream);
  * (kv_heads x K) and v at v_off (kv_heads x V):
  *   q_out (f32 [T, heads*K]), k_out (act [T, kv_heads*K]): RMS norm with eps (whole_row: over all entries of the
  *   projection at once, weight of heads*K resp. kv_heads*K entries; else per head, weight of K entries shared by the
- *   heads; null weight: no norm), then rotation of the first rot_dims entries of each head (entry i with entry
+ *   heads; null weight: no norm, or the weightless one after the rotation, see unit_rms), then rotation of the first rot_dims entries of each head (entry i with entry
  *   i + rot_dims/2) by the angle (pos0 + t) * freq[i], cos and sin multiplied by rot_mult;
  *   v_out (act [T, kv_heads*V]) = (1 - lambda) v + lambda v_first when v_first (act [T, ldvf]) is given; lambda is a
  *   device scalar (act).  Without v_first nothing is written to v_out. */
@@ -363,8 +369,37 @@ typedef struct {
   float* q_out; void* k_out;
   const void* v_first; int ldvf; const void* lambda; void* v_out;
   int T, heads, kv_heads, K, V, act_dtype;
+  int unit_rms;                   /* null norm weights: every head of q and k, after its rotation, divided by its root mean
+                                     square (eps) over K */
 } b2l_seq_qkv_prep_args;
 int b2l_seq_qkv_prep(const b2l_seq_qkv_prep_args* a, b2l_stream_t stream);
+
+/* ---- matrix memory with exponential gates (mLSTM) ----
+ * Per head, from one stacked f32 projection proj [T, ld] (columns at q_off, k_off: heads x K; v_off, g_off: heads x V;
+ * i_off, f_off: heads), with cap(z) = gate_cap * tanh(z / gate_cap):
+ *   log_i = cap(proj_i + b_i);   log_f = log sigmoid(cap(proj_f + b_f))              (b_i, b_f act [heads], may be null)
+ *   m_t = max(log_f + m_(t-1), log_i);   keep = exp(log_f + m_(t-1) - m_t);   put = exp(log_i - m_t)
+ *   S <- keep S + put k v^T;   n <- keep n + put k;   o = S^T (q_mult q) / (max(|n . (q_mult q)|, exp(-m_t)) + den_add)
+ *   out[t, head h] = o / sqrt(mean_V(o^2) + eps) * w_norm[h] * sigmoid(proj_g)        (w_norm act [heads*V], out act)
+ * State per slot, f32, zero at the start: state_S [heads][V][K], state_n [heads][K], state_m [heads].
+ *   b2l_seq_mlstm_step:     everything in one launch, for a single token (T == 1).
+ *   b2l_seq_mlstm_gates:    keep, put and floor = exp(-m_t) (f32 [T, heads] each) of a portion; advances state_m.
+ *   b2l_seq_mlstm_readout:  out from o (f32 [T, ldr]: S^T (q_mult q)) and nq (f32 [T, heads]: n . (q_mult q)) of
+ *                           b2l_seq_scan (decay = keep, vscale = put, ones) and floor. */
+typedef struct {
+  const float* proj; int ld;
+  int q_off, k_off, v_off, g_off, i_off, f_off;
+  const void* b_i; const void* b_f; const void* w_norm;
+  float gate_cap, q_mult, den_add, eps;
+  float* state_S; float* state_n; float* state_m; const int* meta;
+  float* keep; float* put; float* floor;
+  const float* o; int ldr; const float* nq;
+  void* out; int ldo;
+  int T, heads, K, V, act_dtype;
+} b2l_seq_mlstm_args;
+int b2l_seq_mlstm_step(const b2l_seq_mlstm_args* a, b2l_stream_t stream);
+int b2l_seq_mlstm_gates(const b2l_seq_mlstm_args* a, b2l_stream_t stream);
+int b2l_seq_mlstm_readout(const b2l_seq_mlstm_args* a, b2l_stream_t stream);
 
 #ifdef __cplusplus
 }

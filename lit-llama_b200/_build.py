@@ -21,7 +21,7 @@ LIBRARIES = {
     # sequence-mixer kernels: recurrences, local and latent attention, expert routing, f32 residual streams (include/b2l_seq.h)
     "seq": dict(out=os.path.join(PKG, "libb200seq.so"),
                 sources=["seq_api.cu", "seq_elementwise.cu", "seq_scan.cu", "seq_attention.cu", "seq_latent.cu", "seq_moe.cu", "seq_streams.cu",
-                         "seq_depth.cu", "seq_gru.cu", "seq_convrope.cu"]),
+                         "seq_depth.cu", "seq_gru.cu", "seq_convrope.cu", "seq_mlstm.cu"]),
 }
 
 

@@ -17,6 +17,7 @@ from .lugovik import Lugovik, LugovikConfig
 from .zenasun import Zenasun, ZenasunConfig
 from .zuvevik import Zuvevik, ZuvevikConfig
 from .rinirax import Rinirax, RiniraxConfig
+from .lukupel import Lukupel, LukupelConfig
 from .state import SequenceStatePool, StateSpec
 from .engine import Engine
 from .registry import load_model, register
@@ -24,6 +25,6 @@ from .registry import load_model, register
 __all__ = [
     "LLaMA", "LLaMAConfig", "Block", "CausalSelfAttention", "MLP", "RMSNorm", "build_rope_cache", "apply_rope",
     "ColBlockQuantizedLinear", "Linear8bitLt", "find_multiple", "llama_model_lookup", "generate", "sample_probs", "sample_token", "patch_reference", "TPLLaMA", "shard_state_dict",
-    "Lugovik", "LugovikConfig", "Zenasun", "ZenasunConfig", "Zuvevik", "ZuvevikConfig", "Rinirax", "RiniraxConfig",
+    "Lugovik", "LugovikConfig", "Zenasun", "ZenasunConfig", "Zuvevik", "ZuvevikConfig", "Rinirax", "RiniraxConfig", "Lukupel", "LukupelConfig",
     "SequenceStatePool", "StateSpec", "Engine", "load_model", "register",
 ]

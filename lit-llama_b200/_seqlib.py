@@ -8,7 +8,7 @@ import torch
 from . import _build
 
 B2L_BF16, B2L_F32 = 0, 1
-ACT_GELU_TANH, ACT_SILU, ACT_SIGMOID, ACT_CLAMPED_SWISH, ACT_XIELU, ACT_NONE = 0, 1, 2, 3, 4, 5
+ACT_GELU_TANH, ACT_SILU, ACT_SIGMOID, ACT_CLAMPED_SWISH, ACT_XIELU, ACT_NONE, ACT_RELU2 = 0, 1, 2, 3, 4, 5, 6
 NORM_RMS, NORM_LAYER = 0, 1
 SCORE_SOFTMAX, SCORE_SIGMOID = 0, 1
 DECAY_EXP_SOFTPLUS, DECAY_SIGMOID_ROOT = 0, 1
@@ -30,6 +30,7 @@ class ScanArgs(C.Structure):
         ("out", c_void_p), ("ldo", c_int),
         ("T", c_int), ("heads", c_int), ("qk_heads", c_int), ("K", c_int), ("V", c_int), ("act_dtype", c_int),
         ("work_state", c_void_p), ("work_decay", c_void_p), ("n_chunks", c_int),
+        ("ones", c_int), ("state_ones", c_void_p), ("out_ones", c_void_p),
     ]
 
 
@@ -91,15 +92,30 @@ class QkvPrepArgs(C.Structure):
         ("q_out", c_void_p), ("k_out", c_void_p),
         ("v_first", c_void_p), ("ldvf", c_int), ("lambda_", c_void_p), ("v_out", c_void_p),
         ("T", c_int), ("heads", c_int), ("kv_heads", c_int), ("K", c_int), ("V", c_int), ("act_dtype", c_int),
+        ("unit_rms", c_int),
+    ]
+
+
+class MlstmArgs(C.Structure):
+    _fields_ = [
+        ("proj", c_void_p), ("ld", c_int),
+        ("q_off", c_int), ("k_off", c_int), ("v_off", c_int), ("g_off", c_int), ("i_off", c_int), ("f_off", c_int),
+        ("b_i", c_void_p), ("b_f", c_void_p), ("w_norm", c_void_p),
+        ("gate_cap", c_float), ("q_mult", c_float), ("den_add", c_float), ("eps", c_float),
+        ("state_S", c_void_p), ("state_n", c_void_p), ("state_m", c_void_p), ("meta", c_void_p),
+        ("keep", c_void_p), ("put", c_void_p), ("floor", c_void_p),
+        ("o", c_void_p), ("ldr", c_int), ("nq", c_void_p),
+        ("out", c_void_p), ("ldo", c_int),
+        ("T", c_int), ("heads", c_int), ("K", c_int), ("V", c_int), ("act_dtype", c_int),
     ]
 
 
 _SIGS = {
     "b2l_seq_version": (c_int, []),
     "b2l_seq_last_error": (C.c_char_p, []),
-    "b2l_seq_embed": (c_int, [c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "b2l_seq_embed": (c_int, [c_void_p, c_int, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
     "b2l_seq_rmsnorm": (c_int, [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
-    "b2l_seq_norm_add_norm": (c_int, [c_void_p, c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
+    "b2l_seq_norm_add_norm": (c_int, [c_void_p, c_void_p, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
     "b2l_seq_gated_act": (c_int, [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]),
     "b2l_seq_conv_silu": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int,
                                   c_void_p]),
@@ -150,6 +166,9 @@ _SIGS = {
     "b2l_seq_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
     "b2l_seq_depth_step": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float,
                                    c_void_p, c_int, c_int, c_int, c_void_p]),
+    "b2l_seq_mlstm_step": (c_int, [C.POINTER(MlstmArgs), c_void_p]),
+    "b2l_seq_mlstm_gates": (c_int, [C.POINTER(MlstmArgs), c_void_p]),
+    "b2l_seq_mlstm_readout": (c_int, [C.POINTER(MlstmArgs), c_void_p]),
 }
 
 EXPORTS = tuple(_SIGS)

@@ -152,6 +152,7 @@ __device__ __forceinline__ float unary_act(float z, int act, float a, float b) {
     case B2L_SEQ_ACT_GELU_TANH: return gelu_tanh_f(z);
     case B2L_SEQ_ACT_SILU: return silu_f(z);
     case B2L_SEQ_ACT_SIGMOID: return sigmoid_f(z);
+    case B2L_SEQ_ACT_RELU2: { const float r = fmaxf(z, 0.f); return r * r; }
     case B2L_SEQ_ACT_XIELU: return (z > 0.f ? a * z * z : b * expm1_minus_z(fminf(z, 0.f))) + 0.5f * z;
     default: return z;
   }
@@ -249,7 +250,8 @@ extern "C" int b2l_seq_unary_act(const void* in, int ldin, void* out, int ldout,
                                  b2l_stream_t stream) {
   B2L_CHECK_ARG(in && out, "b2l_seq_unary_act: null pointer");
   B2L_CHECK_ARG(T >= 0 && F > 0 && ldin >= F && ldout >= F, "b2l_seq_unary_act: bad size");
-  B2L_CHECK_ARG(act == B2L_SEQ_ACT_GELU_TANH || act == B2L_SEQ_ACT_SILU || act == B2L_SEQ_ACT_SIGMOID || act == B2L_SEQ_ACT_XIELU,
+  B2L_CHECK_ARG(act == B2L_SEQ_ACT_GELU_TANH || act == B2L_SEQ_ACT_SILU || act == B2L_SEQ_ACT_SIGMOID || act == B2L_SEQ_ACT_XIELU ||
+                act == B2L_SEQ_ACT_RELU2,
                 "b2l_seq_unary_act: unknown activation %d", act);
   B2L_CHECK_ARG(act != B2L_SEQ_ACT_XIELU || coef != nullptr, "b2l_seq_unary_act: xIELU without its two coefficients");
   if (T == 0) return 0;

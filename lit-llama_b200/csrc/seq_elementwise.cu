@@ -8,12 +8,16 @@ namespace b2l {
 
 template <typename act_t, typename idx_t>
 __global__ void seq_embed_kernel(const idx_t* __restrict__ tok, const act_t* __restrict__ table, float scale,
-                                 float* __restrict__ x, int D, int vocab) {
+                                 float* __restrict__ x, act_t* __restrict__ h, int D, int vocab) {
   long long t = (long long)tok[blockIdx.x];
   if (t < 0 || t >= vocab) t = 0;
   const act_t* src = table + (size_t)t * D;
   float* dst = x + (size_t)blockIdx.x * D;
-  for (int i = threadIdx.x; i < D; i += blockDim.x) dst[i] = ld_act(src, i) * scale;
+  for (int i = threadIdx.x; i < D; i += blockDim.x) {
+    const float v = ld_act(src, i) * scale;
+    dst[i] = v;
+    if (h) st_act(h, (size_t)blockIdx.x * D + i, v);
+  }
 }
 
 template <typename act_t>
@@ -30,10 +34,10 @@ __global__ void __launch_bounds__(256) seq_rmsnorm_kernel(const float* __restric
   for (int i = threadIdx.x; i < D; i += blockDim.x) st_act(o, i, xr[i] * rinv * ld_act(w, i));
 }
 
-// x += rmsnorm(y) * w_post; optionally h = rmsnorm(x) * w_next.  One CTA per row; the updated row stays in
+// x += mult * rmsnorm(y) * w_post; optionally h = rmsnorm(x) * w_next, or x in the activation type (no w_next).  One CTA per row; the updated row stays in
 // registers between the two passes when it fits (D <= 256 * 8), else it is re-read.
 template <typename act_t>
-__global__ void __launch_bounds__(256) seq_norm_add_norm_kernel(const act_t* __restrict__ y, const act_t* __restrict__ wp, float eps,
+__global__ void __launch_bounds__(256) seq_norm_add_norm_kernel(const act_t* __restrict__ y, const act_t* __restrict__ wp, float eps, float mult,
                                                                 float* __restrict__ x, const act_t* __restrict__ wn,
                                                                 act_t* __restrict__ h, int D) {
   __shared__ float red[32];
@@ -45,12 +49,13 @@ __global__ void __launch_bounds__(256) seq_norm_add_norm_kernel(const act_t* __r
     ss += v * v;
   }
   ss = block_sum(ss, red);
-  const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
+  const float rinv = mult / sqrtf(ss / (float)D + eps);
   float s2 = 0.f;
   for (int i = threadIdx.x; i < D; i += blockDim.x) {
     const float v = xr[i] + ld_act(yr, i) * rinv * ld_act(wp, i);
     xr[i] = v;
     s2 += v * v;
+    if (h && wn == nullptr) st_act(h, (size_t)blockIdx.x * D + i, v);
   }
   if (wn == nullptr) return;
   s2 = block_sum(s2, red);
@@ -62,7 +67,7 @@ __global__ void __launch_bounds__(256) seq_norm_add_norm_kernel(const act_t* __r
 // The same with the row held in registers (D <= 256 * EPT): every operand is requested before the first reduction, so
 // a single-token step pays one memory latency instead of three.
 template <typename act_t, int EPT>
-__global__ void __launch_bounds__(256) seq_norm_add_norm_reg_kernel(const act_t* __restrict__ y, const act_t* __restrict__ wp, float eps,
+__global__ void __launch_bounds__(256) seq_norm_add_norm_reg_kernel(const act_t* __restrict__ y, const act_t* __restrict__ wp, float eps, float mult,
                                                                     float* __restrict__ x, const act_t* __restrict__ wn,
                                                                     act_t* __restrict__ h, int D) {
   __shared__ float red[32];
@@ -82,13 +87,16 @@ __global__ void __launch_bounds__(256) seq_norm_add_norm_reg_kernel(const act_t*
 #pragma unroll
   for (int e = 0; e < EPT; ++e) ss += yv[e] * yv[e];
   ss = block_sum(ss, red);
-  const float rinv = 1.0f / sqrtf(ss / (float)D + eps);
+  const float rinv = mult / sqrtf(ss / (float)D + eps);
   float s2 = 0.f;
 #pragma unroll
   for (int e = 0; e < EPT; ++e) {
     const int i = threadIdx.x + e * 256;
     xv[e] += yv[e] * rinv * pv[e];
-    if (i < D) xr[i] = xv[e];
+    if (i < D) {
+      xr[i] = xv[e];
+      if (h && wn == nullptr) st_act(h, (size_t)blockIdx.x * D + i, xv[e]);
+    }
     s2 += xv[e] * xv[e];
   }
   if (wn == nullptr) return;
@@ -351,16 +359,16 @@ __global__ void seq_headnorm_rope_kernel(const act_t* __restrict__ x, int ldx, c
 
 using namespace b2l;
 
-extern "C" int b2l_seq_embed(const void* tokens, int tokens_i64, const void* table, int act_dtype, float scale, float* x,
+extern "C" int b2l_seq_embed(const void* tokens, int tokens_i64, const void* table, int act_dtype, float scale, float* x, void* h,
                              int T, int D, int vocab, b2l_stream_t stream) {
   B2L_CHECK_ARG(tokens && table && x, "b2l_seq_embed: null pointer");
   B2L_CHECK_ARG(T >= 0 && D > 0 && vocab > 0, "b2l_seq_embed: bad size");
   if (T == 0) return 0;
   B2L_SEQ_DISPATCH(act_dtype, {
     if (tokens_i64)
-      seq_embed_kernel<act_t, long long><<<T, 128, 0, (cudaStream_t)stream>>>((const long long*)tokens, (const act_t*)table, scale, x, D, vocab);
+      seq_embed_kernel<act_t, long long><<<T, 128, 0, (cudaStream_t)stream>>>((const long long*)tokens, (const act_t*)table, scale, x, (act_t*)h, D, vocab);
     else
-      seq_embed_kernel<act_t, int><<<T, 128, 0, (cudaStream_t)stream>>>((const int*)tokens, (const act_t*)table, scale, x, D, vocab);
+      seq_embed_kernel<act_t, int><<<T, 128, 0, (cudaStream_t)stream>>>((const int*)tokens, (const act_t*)table, scale, x, (act_t*)h, D, vocab);
   });
   B2L_LAUNCH_CHECK("seq_embed_kernel");
   return 0;
@@ -376,13 +384,13 @@ extern "C" int b2l_seq_rmsnorm(const float* x, const void* w, float eps, void* o
   return 0;
 }
 
-extern "C" int b2l_seq_norm_add_norm(const void* y, const void* w_post, float eps, float* x, const void* w_next, void* h,
+extern "C" int b2l_seq_norm_add_norm(const void* y, const void* w_post, float eps, float mult, float* x, const void* w_next, void* h,
                                      int T, int D, int act_dtype, b2l_stream_t stream) {
   B2L_CHECK_ARG(y && w_post && x, "b2l_seq_norm_add_norm: null pointer");
-  B2L_CHECK_ARG((w_next == nullptr) == (h == nullptr), "b2l_seq_norm_add_norm: w_next and h go together");
+  B2L_CHECK_ARG(w_next == nullptr || h != nullptr, "b2l_seq_norm_add_norm: a next norm without its output");
   B2L_CHECK_ARG(T >= 0 && D > 0, "b2l_seq_norm_add_norm: bad size");
   if (T == 0) return 0;
-#define B2L_NAN_ARGS (const act_t*)y, (const act_t*)w_post, eps, x, (const act_t*)w_next, (act_t*)h, D
+#define B2L_NAN_ARGS (const act_t*)y, (const act_t*)w_post, eps, mult, x, (const act_t*)w_next, (act_t*)h, D
   B2L_SEQ_DISPATCH(act_dtype, {
     cudaStream_t s_ = (cudaStream_t)stream;
     if (D <= 1024) seq_norm_add_norm_reg_kernel<act_t, 4><<<T, 256, 0, s_>>>(B2L_NAN_ARGS);

@@ -4,7 +4,8 @@
 // A CTA owns one head and a tile of value columns; a column of S (K numbers) lives in the registers of R adjacent
 // lanes (SCAN_KPT numbers each), so a step is R-lane shuffles and no shared-memory traffic for S.  The state is
 // read once, carried through all T tokens of the portion and written once ([V][K] per head, K fastest, so the R
-// lanes of a column read consecutive 16-byte words).  Inputs of SCAN_TC steps are staged in shared memory by the
+// lanes of a column read consecutive 16-byte words).  With `ones` the state has one column more whose value is 1 at every
+// step (a normaliser: the decayed sum of the keys), kept and read out beside the others.  Inputs of SCAN_TC steps are staged in shared memory by the
 // whole CTA with asynchronous copies, one stage ahead of the recurrence.  All arithmetic is f32.
 #include "seq_common.cuh"
 
@@ -49,16 +50,21 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
   const int slot = a.meta[0];
   const bool chunked = a.n_chunks > 1;
   const int t_begin = blockIdx.z * chunk_len, t_end = min(a.T, t_begin + chunk_len);
-  float* st = chunked ? a.work_state + ((size_t)blockIdx.z * a.heads + h) * (size_t)V * K
+  float* st = chunked ? a.work_state + ((size_t)blockIdx.z * a.heads + h) * (size_t)(V + (a.ones ? 1 : 0)) * K
                       : a.state + ((size_t)slot * a.heads + h) * (size_t)V * K;
+  float* st1 = chunked ? st + (size_t)V * K : (a.ones ? a.state_ones + ((size_t)slot * a.heads + h) * (size_t)K : nullptr);   // the column of ones
   const float skip = a.skip ? ld_act((const act_t*)a.skip, h) : 0.f;
   const float* gq = a.q + (size_t)hq * K;
   const float* gk = a.k + (size_t)hq * K;
   const float* gv = a.v + (size_t)h * V + v0;
   const float* gd = a.decay + (a.decay_per_channel ? (size_t)h * K : (size_t)h);
-  const int ncol = min(cols, V - v0);
+  const int VT = V + (a.ones ? 1 : 0);         // state columns
+  const int ncol = min(cols, VT - v0);         // ... of this CTA
+  const int nval = min(ncol, V - v0);          // ... of which values (the column of ones is the last of all)
+  const bool warp_live = (tid & ~31) / R < ncol;   // a warp whose column groups all lie past the last column has nothing to compute
 
-  // padding that no copy ever touches: q = k = 0 and d = 1 beyond K, v = 0 beyond V, vs = 1 without a value scale
+  // padding that no copy ever touches: q = k = 0 and d = 1 beyond K, v = 1 in the column of ones and 0 beyond it, vs = 1
+  // without a value scale
   for (int b = 0; b < 2; ++b) {
     float* sq = smem + b * stage;
     float* sk = sq + SCAN_TC * KP;
@@ -73,7 +79,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
       }
     }
     for (int i = tid; i < SCAN_TC * cols; i += SCAN_THREADS)
-      if (i % cols >= ncol) sv[i] = 0.f;
+      if (i % cols >= nval) sv[i] = i % cols < ncol ? 1.f : 0.f;
     if (tid < SCAN_TC) svs[tid] = 1.f;
   }
 
@@ -100,8 +106,8 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
         if (a.decay_per_channel) cp_async4(sd + t * KP + kk, gd + (size_t)(t0 + t) * a.ldd + kk);
       }
     }
-    for (int i = tid; i < nt * ncol; i += SCAN_THREADS) {
-      const int t = i / ncol, c = i - t * ncol;
+    for (int i = tid; i < nt * nval; i += SCAN_THREADS) {
+      const int t = i / nval, c = i - t * nval;
       cp_async4(sv + t * cols + c, gv + (size_t)(t0 + t) * a.ldv + c);
     }
     if (tid < nt) {
@@ -121,7 +127,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
 #pragma unroll
     for (int i = 0; i < SCAN_KPT; ++i) {
       const int kk = ((i >> 2) * R + r) * 4 + (i & 3);
-      S[j][i] = (PASS == 0 && kk < K && vcol < V) ? st[(size_t)vcol * K + kk] : 0.f;
+      S[j][i] = (PASS == 0 && kk < K && vcol < VT) ? (vcol < V ? st[(size_t)vcol * K + kk] : st1[kk]) : 0.f;
     }
   }
   float P[PASS ? SCAN_KPT : 1];       // PASS 1: the chunk's total decay of this lane's key channels
@@ -153,7 +159,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
     const float* sb = svs + SCAN_TC;
 
 #pragma unroll(DELTA ? 2 : 1)
-    for (int t = 0; t < nt; ++t) {
+    for (int t = 0; t < (warp_live ? nt : 0); ++t) {
       const float4* q4 = reinterpret_cast<const float4*>(sq + t * KP);
       const float4* k4 = reinterpret_cast<const float4*>(sk + t * KP);
       float kr[SCAN_KPT], qr[SCAN_KPT];
@@ -258,7 +264,8 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
     if (PASS == 0) {
       for (int i = tid; i < nt * ncol; i += SCAN_THREADS) {
         const int t = i / ncol, c = i - t * ncol;
-        a.out[(size_t)(t0 + t) * a.ldo + (size_t)h * V + v0 + c] = so[t * cols + c];
+        if (c < nval) a.out[(size_t)(t0 + t) * a.ldo + (size_t)h * V + v0 + c] = so[t * cols + c];
+        else a.out_ones[(size_t)(t0 + t) * a.heads + h] = so[t * cols + c];
       }
     }
     if (DELTA && more && tid < SCAN_TC) smem[(b ^ 1) * stage + beta_at + tid] = sigmoid_f(beta_next);
@@ -271,7 +278,7 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
 #pragma unroll
     for (int i = 0; i < SCAN_KPT; ++i) {
       const int kk = ((i >> 2) * R + r) * 4 + (i & 3);
-      if (kk < K && vcol < V) st[(size_t)vcol * K + kk] = S[j][i];
+      if (kk < K && vcol < VT) (vcol < V ? st[(size_t)vcol * K + kk] : st1[kk]) = S[j][i];
     }
   }
   if (PASS && blockIdx.x == 0 && cidx == 0) {
@@ -291,12 +298,14 @@ __global__ void __launch_bounds__(SCAN_THREADS, DELTA ? 2 : 3) seq_scan_kernel(b
 // Between the passes of a chunked portion: work_state[c] (a chunk's local end state) becomes the chunk's START state,
 // s_0 = the slot's state, s_(c+1) = D_c s_c + local_c, and the slot's state becomes s_n.  One thread per state entry.
 __global__ void seq_scan_combine_kernel(b2l_seq_scan_args a) {
-  const size_t per_head = (size_t)a.V * a.K, n = (size_t)a.heads * per_head;
+  const size_t per_head = (size_t)(a.V + (a.ones ? 1 : 0)) * a.K, n = (size_t)a.heads * per_head, n_val = (size_t)a.V * a.K;
   const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const int h = (int)(i / per_head), kk = (int)(i % a.K);
-  float* st = a.state + (size_t)a.meta[0] * n;
-  float s = st[i];
+  const size_t in_head = i % per_head;
+  float* st = in_head < n_val ? a.state + ((size_t)a.meta[0] * a.heads + h) * n_val + in_head
+                              : a.state_ones + ((size_t)a.meta[0] * a.heads + h) * a.K + (in_head - n_val);
+  float s = *st;
   const size_t dstep = (size_t)a.heads * (a.decay_per_channel ? a.K : 1);
   const float* dp = a.work_decay + (size_t)h * (a.decay_per_channel ? a.K : 1) + (a.decay_per_channel ? kk : 0);
   for (int c0 = 0; c0 < a.n_chunks; c0 += 8) {        // eight chunks' operands are requested together
@@ -313,7 +322,7 @@ __global__ void seq_scan_combine_kernel(b2l_seq_scan_args a) {
       s = fmaf(d[u], s, local[u]);
     }
   }
-  st[i] = s;
+  *st = s;
 }
 
 static DynSmemCache g_scan_smem[10];
@@ -337,7 +346,9 @@ extern "C" int b2l_seq_scan(const b2l_seq_scan_args* a, b2l_stream_t stream) {
   B2L_CHECK_SUPPORTED(a->K <= 32 * SCAN_KPT, "b2l_seq_scan: key size %d above %d", a->K, 32 * SCAN_KPT);
   B2L_CHECK_ARG(a->n_chunks <= 1 || (!a->delta && a->work_state && a->work_decay && a->n_chunks == (a->T + SCAN_CHUNK - 1) / SCAN_CHUNK),
                 "b2l_seq_scan: chunked portions need the workspace, no delta rule and n_chunks from b2l_seq_scan_chunks");
+  B2L_CHECK_ARG(!a->ones || (a->state_ones && a->out_ones && !a->skip && !a->delta), "b2l_seq_scan: the column of ones needs its state and its output, no skip and no delta rule");
   if (a->T == 0) return 0;
+  const int VT = a->V + (a->ones ? 1 : 0);
   const int n_chunks = a->n_chunks > 1 ? a->n_chunks : 1;
   const int chunk_len = n_chunks > 1 ? SCAN_CHUNK : a->T;
   int R = 1;
@@ -349,7 +360,7 @@ extern "C" int b2l_seq_scan(const b2l_seq_scan_args* a, b2l_stream_t stream) {
   auto al16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
   const int vec = a->K % 4 == 0 && a->ldq % 4 == 0 && a->ldk % 4 == 0 && al16(a->q) && al16(a->k) &&
                   (!a->decay_per_channel || (a->ldd % 4 == 0 && al16(a->decay)));
-  dim3 grid((unsigned)((a->V + cols - 1) / cols), (unsigned)a->heads, (unsigned)n_chunks);
+  dim3 grid((unsigned)((VT + cols - 1) / cols), (unsigned)a->heads, (unsigned)n_chunks);
   cudaStream_t s = (cudaStream_t)stream;
 #define B2L_SCAN_LAUNCH(D, T_, P_, C_, slot_)                                                 \
   do {                                                                                        \
@@ -366,7 +377,7 @@ extern "C" int b2l_seq_scan(const b2l_seq_scan_args* a, b2l_stream_t stream) {
     if (cpl == 2) { if (bf) B2L_SCAN_LAUNCH(0, __nv_bfloat16, 1, 2, 4); else B2L_SCAN_LAUNCH(0, float, 1, 2, 5); }
     else { if (bf) B2L_SCAN_LAUNCH(0, __nv_bfloat16, 1, 1, 6); else B2L_SCAN_LAUNCH(0, float, 1, 1, 7); }
     B2L_LAUNCH_CHECK("seq_scan_kernel (local states)");
-    const size_t n = (size_t)a->heads * a->V * a->K;
+    const size_t n = (size_t)a->heads * VT * a->K;
     seq_scan_combine_kernel<<<(unsigned)((n + 255) / 256), 256, 0, s>>>(*a);
     B2L_LAUNCH_CHECK("seq_scan_combine_kernel");
   }

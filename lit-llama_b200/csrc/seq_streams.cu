@@ -137,7 +137,9 @@ __global__ void seq_scale_kernel(float* __restrict__ z, size_t n, float mult) {
 // Attention operands of one token from the stacked projection row, one CTA per token.
 //   q_out (f32) and k_out (act): RMS norm (whole_row: over all heads*K entries with a weight of that size; else per
 //   head with a weight of K entries shared by the heads; no weight: no norm), then rotation of the first rot_dims
-//   entries of every head (entry i with entry i + rot_dims/2) by the angle (pos0 + t) * freq[i].
+//   entries of every head (entry i with entry i + rot_dims/2) by the angle (pos0 + t) * freq[i]; unit_rms (no weights): the
+//   rotated head divided by its root mean square.  A rotation keeps the length of the pairs it turns up to rot_mult, so
+//   the sum of squares is taken from the entries before it.
 //   v_out (act): (1 - lambda) v + lambda v_first when v_first is given (lambda read on the device), else not written.
 template <typename act_t>
 __global__ void __launch_bounds__(256) seq_qkv_prep_kernel(b2l_seq_qkv_prep_args a) {
@@ -164,10 +166,11 @@ __global__ void __launch_bounds__(256) seq_qkv_prep_kernel(b2l_seq_qkv_prep_args
       const act_t* p = x + (size_t)hd * K;
       const act_t* wh = w ? (a.whole_row ? w + (size_t)hd * K : w) : nullptr;
       float r = r_row;
-      if (w && !a.whole_row) {
+      if (a.unit_rms || (w && !a.whole_row)) {
+        const float turned = a.unit_rms ? a.rot_mult : 1.f;
         float ss = 0.f;
         for (int i = lane; i < K; i += 32) {
-          const float v = ld_act(p, i);
+          const float v = ld_act(p, i) * (i < a.rot_dims ? turned : 1.f);
           ss += v * v;
         }
         ss = warp_sum(ss);
@@ -294,6 +297,7 @@ extern "C" int b2l_seq_qkv_prep(const b2l_seq_qkv_prep_args* a, b2l_stream_t str
   B2L_CHECK_ARG(a->T >= 0 && a->heads > 0 && a->kv_heads > 0 && a->K > 0 && a->V > 0, "b2l_seq_qkv_prep: bad size");
   B2L_CHECK_ARG(a->rot_dims >= 0 && a->rot_dims <= a->K && a->rot_dims % 2 == 0 && (a->rot_dims == 0 || a->freq), "b2l_seq_qkv_prep: bad rotation");
   B2L_CHECK_ARG((a->v_first == nullptr) || (a->v_out && a->lambda), "b2l_seq_qkv_prep: value mixing needs lambda and an output");
+  B2L_CHECK_ARG(!a->unit_rms || (a->q_norm == nullptr && a->k_norm == nullptr), "b2l_seq_qkv_prep: the norm after the rotation has no weight");
   if (a->T == 0) return 0;
   B2L_SEQ_DISPATCH(a->act_dtype, (seq_qkv_prep_kernel<act_t><<<a->T, 256, 0, (cudaStream_t)stream>>>(*a)));
   B2L_LAUNCH_CHECK("seq_qkv_prep_kernel");

@@ -127,7 +127,7 @@ class Lugovik:
         if self.dtype == torch.float32 and torch.backends.cuda.matmul.allow_tf32:
             raise RuntimeError("float32 models need true 32-bit products: torch.backends.cuda.matmul.allow_tf32 is on")
         x = torch.empty((T, D), dtype=torch.float32, device=dev)
-        S.check(lib.b2l_seq_embed(_p(tokens), int(tokens.dtype == torch.int64), _p(self.embed), ctx.act, self.config.embedding_scale, _p(x), T, D,
+        S.check(lib.b2l_seq_embed(_p(tokens), int(tokens.dtype == torch.int64), _p(self.embed), ctx.act, self.config.embedding_scale, _p(x), None, T, D,
                                   self.vocab, ctx.stream), "b2l_seq_embed")
         h = torch.empty((T, D), dtype=self.dtype, device=dev)
         if self.layers:
@@ -136,11 +136,11 @@ class Lugovik:
             nxt = self.layers[i + 1].norm1 if i + 1 < len(self.layers) else None
             y = layer.mixer.forward(h, ctx)
             after = layer.norm2 if layer.mlp is not None else nxt
-            S.check(lib.b2l_seq_norm_add_norm(_p(y), _p(layer.norm1b), self.eps, _p(x), _p(after), _p(h) if after is not None else None, T, D,
+            S.check(lib.b2l_seq_norm_add_norm(_p(y), _p(layer.norm1b), self.eps, 1.0, _p(x), _p(after), _p(h) if after is not None else None, T, D,
                                               ctx.act, ctx.stream), "b2l_seq_norm_add_norm")
             if layer.mlp is not None:
                 y = layer.mlp.forward(h, ctx)
-                S.check(lib.b2l_seq_norm_add_norm(_p(y), _p(layer.norm2b), self.eps, _p(x), _p(nxt), _p(h) if nxt is not None else None, T, D,
+                S.check(lib.b2l_seq_norm_add_norm(_p(y), _p(layer.norm2b), self.eps, 1.0, _p(x), _p(nxt), _p(h) if nxt is not None else None, T, D,
                                                   ctx.act, ctx.stream), "b2l_seq_norm_add_norm")
             if self.capture_layers is not None:
                 self.capture_layers.append(x.clone())

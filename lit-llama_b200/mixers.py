@@ -13,22 +13,27 @@ constants are constructor parameters.
     RetentionMixer       linear attention with a fixed decay per head, rotated q / k, per-head unit-RMS read-out, silu gate
     MoEFeedForward       routed gated experts: softmax or sigmoid scores, selection bias, expert groups, top-k, identity
                          experts, weights renormalised or not, on an expert's output or on its input, clamped gated unit
-    SlidingWindowAttention  causal softmax attention over the last `window` positions: q/k norm over the whole projection
-                         or per head, partial rotation, grouped kv heads, values mixed with an earlier layer's, a sigmoid
-                         gate per output channel, ring cache of `window` positions
+    LocalAttention       causal softmax attention over the last `window` positions (SlidingWindowAttention) or inside blocks:
+                         q/k norm over the whole projection or per head before the rotation, or weightless per head after it,
+                         partial rotation, grouped kv heads, values mixed with an earlier layer's, an optional sigmoid gate per
+                         output channel, ring cache of one window or block
     PairHashEmbedding    token embedding plus a hashed (previous token, token) embedding, into several residual streams
     HyperConnection      one sublayer's read weights, stream-mixing matrix and write weights over several residual streams
-    DenseMLP             W_down act(W_up h) without a gate: gelu_tanh, silu, or xIELU with its two learned numbers
+    DenseMLP             W_down act(W_up h) without a gate: gelu_tanh, silu, relu2, or xIELU with its two learned numbers
     DifferentialAttention  causal softmax attention with two score maps per head over the same values, combined as
                          a0 - lambda a1 and divided by its root mean square; biases and short convolutions on q / k / v,
                          interleaved rotation, grouped kv heads, keys and values of its own or of an earlier layer
     MinGRUMixer          S_t = (1 - z_t) S_(t-1) + z_t c_t per channel with gates that read only the current token, silu gate
     DepthAverage         the residual step of layers whose input is a learned average over all earlier layers' results
+    MatrixMemoryMixer    mLSTM: a matrix state per head with exponential input gates, sigmoid forget gates, a normaliser and a
+                         running maximum; per-head unit-RMS read-out, one weight, a sigmoid gate per channel
+    share_weights        the same mixer over the same weights with a state of its own (a layer that runs again)
 
 A mixer is built from a dict of weight tensors (`from_weights`) and runs one portion of one sequence:
 `forward(h, ctx)` with h [T, width] in the model's activation dtype.  Products go through torch (cuBLAS), as the
 dense linears of the package's LLaMA do; everything else is a kernel of libb200seq.  What a mixer carries between
 tokens is declared by `state_specs()` and lives in a `SequenceStatePool`.  CUDA only; no CPU fallback."""
+import copy
 import ctypes as C
 import math
 from typing import Dict, List, Optional, Tuple
@@ -83,6 +88,16 @@ def stack_rows(parts: List[torch.Tensor]) -> Tuple[torch.Tensor, List[int]]:
     return torch.cat(rows, dim=0).contiguous(), offs
 
 
+def share_weights(mixer, name: str):
+    """`mixer` over the same weight tensors with a state of its own under `name`, for a layer that uses another layer's
+    weights.  Mixers find their state by their name and hold everything else in tensors they never write."""
+    if hasattr(mixer, "branches"):
+        raise ValueError("a mixer of several branches has several states: share its branches one by one")
+    twin = copy.copy(mixer)
+    twin.name = name
+    return twin
+
+
 def linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return F.linear(x, w)
 
@@ -116,10 +131,10 @@ class GatedMLP:
 
 
 class DenseMLP:
-    """W_down act(W_up h), no gate.  act: gelu_tanh, silu, sigmoid, or xIELU with its two learned numbers `params` = (p, q):
+    """W_down act(W_up h), no gate.  act: gelu_tanh, silu, sigmoid, relu2 (max(z, 0)^2), or xIELU with its two learned numbers `params` = (p, q):
     softplus(p) z^2 + z/2 for z > 0, (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2 otherwise."""
 
-    ACTS = {"gelu_tanh": S.ACT_GELU_TANH, "silu": S.ACT_SILU, "sigmoid": S.ACT_SIGMOID, "xielu": S.ACT_XIELU}
+    ACTS = {"gelu_tanh": S.ACT_GELU_TANH, "silu": S.ACT_SILU, "sigmoid": S.ACT_SIGMOID, "relu2": S.ACT_RELU2, "xielu": S.ACT_XIELU}
 
     def __init__(self, up: torch.Tensor, down: torch.Tensor, act: str = "gelu_tanh", params: Optional[torch.Tensor] = None) -> None:
         if act not in self.ACTS:
@@ -147,17 +162,18 @@ class DenseMLP:
 
 # ------------------------------------------------------------------------------------------------ recurrences
 def _scan(ctx: StepContext, *, q, ldq, k, ldk, v, ldv, q_mult, decay, ldd, per_channel, state, out, ldo, heads, qk_heads,
-          K, V, beta=None, ldb=0, vscale=None, ldvs=0, skip=None) -> None:
+          K, V, beta=None, ldb=0, vscale=None, ldvs=0, skip=None, state_ones=None, out_ones=None) -> None:
     lib = S.lib()
     n_chunks = lib.b2l_seq_scan_chunks(ctx.T, int(beta is not None))
     ws = wd = None
     if n_chunks > 1:      # long portion, no delta rule: chunks in parallel (local states, combine, outputs)
-        ws = torch.empty((n_chunks, heads, V, K), dtype=torch.float32, device=state.device)
+        ws = torch.empty((n_chunks, heads, V + int(state_ones is not None), K), dtype=torch.float32, device=state.device)
         wd = torch.empty((n_chunks, heads, K if per_channel else 1), dtype=torch.float32, device=state.device)
     a = S.ScanArgs(q=q, ldq=ldq, k=k, ldk=ldk, v=v, ldv=ldv, q_mult=float(q_mult), decay=decay, ldd=ldd,
                    decay_per_channel=int(per_channel), beta=beta, ldb=ldb, delta=int(beta is not None), vscale=vscale, ldvs=ldvs,
                    skip=skip, state=_p(state), meta=_p(ctx.meta), out=out, ldo=ldo, T=ctx.T, heads=heads, qk_heads=qk_heads, K=K, V=V,
-                   act_dtype=ctx.act, work_state=_p(ws), work_decay=_p(wd), n_chunks=n_chunks)
+                   act_dtype=ctx.act, work_state=_p(ws), work_decay=_p(wd), n_chunks=n_chunks, ones=int(state_ones is not None), state_ones=_p(state_ones),
+                   out_ones=out_ones)
     S.check(lib.b2l_seq_scan(C.byref(a), ctx.stream), "b2l_seq_scan")
 
 
@@ -253,6 +269,63 @@ class Mamba2Mixer:
         return linear(out, self.w_o)
 
 
+class MatrixMemoryMixer:
+    """Matrix memory with exponential gates (mLSTM), per head, cap(z) = gate_cap tanh(z / gate_cap):
+
+        q = W_q h dim^-1/2;  k = W_k h;  v = W_v h;  log_i = cap(W_i h + b_i);  log_f = log sigmoid(cap(W_f h + b_f))
+        m <- max(log_f + m, log_i), starting at 0;  keep = exp(log_f + m_before - m);  put = exp(log_i - m)
+        S <- keep S + put k v^T;  n <- keep n + put k;  o = S^T q / (max(|n . q|, exp(-m)) + DEN_ADD)
+        y = W_o (o / rms(o) * w_norm * sigmoid(W_g h))
+    The projections are one product whose f32 accumulator is kept; everything up to the read-out is f32.  A single token is
+    one launch; a portion runs gates, scan (n is a column of ones beside the values) and read-out.  State per sequence:
+    S (heads x vdim x dim), n (heads x dim), m (heads), all f32, zero at the start."""
+
+    DEN_ADD = 1e-6
+
+    def __init__(self, name: str, W: Dict[str, torch.Tensor], p: str, *, heads: int, dim: int, vdim: int, gate_cap: float, eps: float) -> None:
+        self.name, self.H, self.K, self.V, self.gate_cap, self.eps = name, int(heads), int(dim), int(vdim), float(gate_cap), float(eps)
+        parts = [W[p + n] for n in ("q", "k", "v", "g", "i", "f")]
+        want = [self.H * self.K] * 2 + [self.H * self.V] * 2 + [self.H] * 2
+        assert [w.shape[0] for w in parts] == want and W[p + "o"].shape[1] == self.H * self.V, "matrix memory: projections do not fit the head sizes"
+        self.w_in, (self.o_q, self.o_k, self.o_v, self.o_g, self.o_i, self.o_f) = stack_rows(parts)
+        self.b_i, self.b_f = W[p + "i.b"].contiguous(), W[p + "f.b"].contiguous()
+        self.w_norm, self.w_o = W[p + "norm"].contiguous(), W[p + "o"].contiguous()
+
+    def state_specs(self) -> Dict[str, StateSpec]:
+        return {self.name + ".S": StateSpec((self.H, self.V, self.K), torch.float32),
+                self.name + ".n": StateSpec((self.H, self.K), torch.float32),
+                self.name + ".m": StateSpec((self.H,), torch.float32)}
+
+    def args(self, proj: torch.Tensor, out: torch.Tensor, ctx: StepContext) -> "S.MlstmArgs":
+        st, n = ctx.state, self.name
+        return S.MlstmArgs(proj=_p(proj), ld=proj.shape[1], q_off=self.o_q, k_off=self.o_k, v_off=self.o_v, g_off=self.o_g, i_off=self.o_i,
+                           f_off=self.o_f, b_i=_p(self.b_i), b_f=_p(self.b_f), w_norm=_p(self.w_norm), gate_cap=self.gate_cap, q_mult=self.K ** -0.5,
+                           den_add=self.DEN_ADD, eps=self.eps, state_S=_p(st[n + ".S"]), state_n=_p(st[n + ".n"]), state_m=_p(st[n + ".m"]),
+                           meta=_p(ctx.meta), out=_p(out), ldo=out.shape[1], T=ctx.T, heads=self.H, K=self.K, V=self.V, act_dtype=ctx.act)
+
+    def recur(self, proj: torch.Tensor, out: torch.Tensor, ctx: StepContext) -> None:
+        """Everything between the input product and the output product."""
+        lib, T, dev, H, ld = S.lib(), ctx.T, out.device, self.H, proj.shape[1]
+        a = self.args(proj, out, ctx)
+        if T == 1:
+            S.check(lib.b2l_seq_mlstm_step(C.byref(a), ctx.stream), "b2l_seq_mlstm_step")
+            return
+        gates = torch.empty((4, T, H), dtype=torch.float32, device=dev)               # keep, put, exp(-m), n . q
+        o = torch.empty((T, H * self.V), dtype=torch.float32, device=dev)
+        a.keep, a.put, a.floor, a.nq, a.o, a.ldr = _p(gates[0]), _p(gates[1]), _p(gates[2]), _p(gates[3]), _p(o), H * self.V
+        S.check(lib.b2l_seq_mlstm_gates(C.byref(a), ctx.stream), "b2l_seq_mlstm_gates")
+        _scan(ctx, q=_p(proj, self.o_q), ldq=ld, k=_p(proj, self.o_k), ldk=ld, v=_p(proj, self.o_v), ldv=ld, q_mult=self.K ** -0.5, decay=a.keep, ldd=H,
+              per_channel=False, vscale=a.put, ldvs=H, state=ctx.state[self.name + ".S"], out=a.o, ldo=H * self.V, heads=H, qk_heads=H, K=self.K,
+              V=self.V, state_ones=ctx.state[self.name + ".n"], out_ones=a.nq)
+        S.check(lib.b2l_seq_mlstm_readout(C.byref(a), ctx.stream), "b2l_seq_mlstm_readout")
+
+    def forward(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        proj = linear_f32(h, self.w_in)
+        out = torch.empty((ctx.T, self.H * self.V), dtype=h.dtype, device=h.device)
+        self.recur(proj, out, ctx)
+        return linear(out, self.w_o)
+
+
 class MinGRUMixer:
     """A gated recurrence whose gates read only the current token, channel by channel:
 
@@ -287,14 +360,17 @@ class MinGRUMixer:
 
 # ------------------------------------------------------------------------------------------------ rotation
 def rope_frequencies(dims: int, base: float, scaling: Optional[dict]) -> Tuple[torch.Tensor, float]:
-    """Per-pair rotation frequencies f_i = base^(-2i/dims), i < dims/2, optionally YaRN-scaled: with
+    """Per-pair rotation frequencies f_i = base^(-2i/dims), i < dims/2, optionally scaled.  Linear (scaling has a `factor`
+    alone): f_i / factor.  YaRN (it also has `original`, `fast` and `slow`): with
     d(t) = dims ln(original / (2 pi t)) / (2 ln base), lo = max(floor(d(fast)), 0), hi = min(ceil(d(slow)), dims - 1) and
     ramp_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) the frequency becomes f_i / factor * ramp_i + f_i (1 - ramp_i),
     and cos / sin are multiplied by 0.1 ln(factor) + 1.  Returns (f32 frequencies on the CPU, multiplier)."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     f = float(base) ** (-2.0 * i / dims)
     mult = 1.0
-    if scaling:
+    if scaling and "original" not in scaling:
+        f = f / float(scaling["factor"])
+    elif scaling:
         factor, orig = float(scaling["factor"]), float(scaling["original"])
 
         def d(t: float) -> float:
@@ -443,33 +519,44 @@ class ParallelMixer:
         return linear(out, self.w_o)
 
 
-class SlidingWindowAttention:
-    """Causal softmax attention over the last `window` positions (the query's own and the window - 1 before it).
+class LocalAttention:
+    """Causal softmax attention over the last `window` positions (the query's own and the window - 1 before it), over the
+    query's block of `block` positions (query p sees j <= p with j // block == p // block), or, with neither, over the whole
+    sequence up to `max_positions`.
 
         q, k, v = W_q h, W_k h, W_v h (one stacked product, with the gate);  q, k: RMS norm, over the whole projection
         with a weight of its size (`norm_over` = "row") or per head with one weight of `dim` entries ("head"), then
-        rotation of the first rot.dims entries of every head (entry i with entry i + dims/2)
+        rotation of the first rot.dims entries of every head (entry i with entry i + dims/2); or ("unit") the rotation first,
+        then every head divided by its root mean square, without a weight
         v <- (1 - lambda) v + lambda v_first in every layer with `v_mix` but the first of them, whose v is v_first
         weights = softmax(q . k * scale) over the visible keys (ordinary softmax, no sink); query head h reads
         key / value head h // (heads / kv_heads)
-        y = W_o (concat_h(sum_j weight_j v_j) * sigmoid(W_g h))            a gate per output channel
+        y = W_o (concat_h(sum_j weight_j v_j) * sigmoid(W_g h))            a gate per output channel; no gate when not `gate`
 
-    State per sequence: a ring of `window` positions of rotated keys and (mixed) values, entry position % window.  The
-    first value-mixing layer of a step leaves its values in `ctx.shared` for the later ones."""
+    State per sequence: a ring of `window` (or `block`) positions of rotated keys and (mixed) values, entry position %
+    size.  The first value-mixing layer of a step leaves its values in `ctx.shared` for the later ones."""
 
-    def __init__(self, name: str, W: Dict[str, torch.Tensor], p: str, *, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int,
-                 eps: float, rot: Optional[dict] = None, v_mix: bool = False, norm_over: str = "row", mix_key: str = "v_first") -> None:
+    NORMS = ("row", "head", "unit")
+
+    def __init__(self, name: str, W: Dict[str, torch.Tensor], p: str, *, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float,
+                 window: Optional[int] = None, block: Optional[int] = None, max_positions: int = 0, rot: Optional[dict] = None,
+                 norm_over: str = "row", gate: bool = True, v_mix: bool = False, mix_key: str = "v_first") -> None:
         self.name, self.H, self.G, self.K, self.V, self.scale, self.eps = name, int(heads), int(kv_heads), int(dim), int(vdim), float(scale), eps
-        self.window = int(window)
-        if self.window < 1 or self.H % self.G:
-            raise ValueError("sliding-window attention: the window must hold at least the query's own position, heads a multiple of kv_heads")
-        if norm_over not in ("row", "head"):
-            raise ValueError(f"sliding-window attention: norm over {norm_over!r}")
-        self.whole_row, self.v_mix, self.mix_key = int(norm_over == "row"), bool(v_mix), mix_key
+        if window is not None and block is not None:
+            raise ValueError("local attention: a window or blocks, not both")
+        self.window = 0 if window is None else int(window)                     # 0: inside blocks
+        self.ring = int(window if window is not None else (block or max_positions))
+        if self.ring < 1 or self.H % self.G:
+            raise ValueError("local attention: the window or block must hold at least the query's own position, heads a multiple of kv_heads")
+        if norm_over not in self.NORMS:
+            raise ValueError(f"local attention: norm over {norm_over!r}")
+        self.whole_row, self.unit_rms, self.v_mix, self.mix_key = int(norm_over == "row"), int(norm_over == "unit"), bool(v_mix), mix_key
         assert W[p + "q"].shape[0] == heads * dim and W[p + "k"].shape[0] == kv_heads * dim and W[p + "v"].shape[0] == kv_heads * vdim, \
-            "sliding-window attention: projections do not fit the head sizes"
-        assert W[p + "g"].shape[0] == heads * vdim and W[p + "o"].shape[1] == heads * vdim, "sliding-window attention: gate / output do not fit"
-        self.w_in, (self.o_q, self.o_k, self.o_v, self.o_g) = stack_rows([W[p + "q"], W[p + "k"], W[p + "v"], W[p + "g"]])
+            "local attention: projections do not fit the head sizes"
+        assert W[p + "o"].shape[1] == heads * vdim and (not gate or W[p + "g"].shape[0] == heads * vdim), "local attention: gate / output do not fit"
+        self.w_in, offs = stack_rows([W[p + "q"], W[p + "k"], W[p + "v"]] + ([W[p + "g"]] if gate else []))
+        self.o_q, self.o_k, self.o_v = offs[:3]
+        self.o_g = offs[3] if gate else None
         self.q_norm = W[p + "q.norm"].contiguous() if (p + "q.norm") in W else None
         self.k_norm = W[p + "k.norm"].contiguous() if (p + "k.norm") in W else None
         self.lam = W[p + "vmix"].reshape(1).contiguous() if self.v_mix else None
@@ -482,8 +569,8 @@ class SlidingWindowAttention:
 
     def state_specs(self) -> Dict[str, StateSpec]:
         dt = self.w_o.dtype
-        return {self.name + ".k": StateSpec((self.window, self.G, self.K), dt, zero_on_acquire=False),
-                self.name + ".v": StateSpec((self.window, self.G, self.V), dt, zero_on_acquire=False)}
+        return {self.name + ".k": StateSpec((self.ring, self.G, self.K), dt, zero_on_acquire=False),
+                self.name + ".v": StateSpec((self.ring, self.G, self.V), dt, zero_on_acquire=False)}
 
     def forward(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         lib, T, dev = S.lib(), ctx.T, h.device
@@ -505,15 +592,27 @@ class SlidingWindowAttention:
                           whole_row=self.whole_row, eps=self.eps, freq=_p(self.freq), rot_dims=self.rot_dims, rot_mult=self.rot_mult,
                           meta=_p(ctx.meta), q_out=_p(q), k_out=_p(kn), v_first=_p(first[0], first[1]) if first is not None else None,
                           ldvf=first[2] if first is not None else 0, lambda_=_p(self.lam) if first is not None else None, v_out=_p(vm), T=T,
-                          heads=self.H, kv_heads=self.G, K=self.K, V=self.V, act_dtype=ctx.act)
+                          heads=self.H, kv_heads=self.G, K=self.K, V=self.V, act_dtype=ctx.act, unit_rms=self.unit_rms)
         S.check(lib.b2l_seq_qkv_prep(C.byref(a), ctx.stream), "b2l_seq_qkv_prep")
         att = torch.empty((T, self.H * self.V), dtype=h.dtype, device=dev)
+        gated = self.o_g is not None
         b = S.AttnArgs(q=_p(q), k_new=_p(kn), v_new=_p(v, v_off), ldv=ldv, cache_k=_p(ctx.state[self.name + ".k"]),
-                       cache_v=_p(ctx.state[self.name + ".v"]), meta=_p(ctx.meta), gate=_p(proj, self.o_g), ldg=ld, out=_p(att), ldo=self.H * self.V,
-                       scale=self.scale, softcap=0.0, out_mult=1.0, has_sink=0, block=self.window, T=T, heads=self.H, kv_heads=self.G, K=self.K,
-                       V=self.V, act_dtype=ctx.act, window=self.window, gate_per_channel=1)
+                       cache_v=_p(ctx.state[self.name + ".v"]), meta=_p(ctx.meta), gate=_p(proj, self.o_g) if gated else None, ldg=ld if gated else 0,
+                       out=_p(att), ldo=self.H * self.V, scale=self.scale, softcap=0.0, out_mult=1.0, has_sink=0, block=self.ring, T=T, heads=self.H,
+                       kv_heads=self.G, K=self.K, V=self.V, act_dtype=ctx.act, window=self.window, gate_per_channel=int(gated))
         local_attention(b, ctx)
         return linear(att, self.w_o)
+
+
+class SlidingWindowAttention(LocalAttention):
+    """`LocalAttention` over a sliding window, q / k norms with weights, the output gated per channel."""
+
+    def __init__(self, name: str, W: Dict[str, torch.Tensor], p: str, *, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, window: int,
+                 eps: float, rot: Optional[dict] = None, v_mix: bool = False, norm_over: str = "row", mix_key: str = "v_first") -> None:
+        if norm_over not in ("row", "head"):
+            raise ValueError(f"sliding-window attention: norm over {norm_over!r}")
+        super().__init__(name, W, p, heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, scale=scale, eps=eps, window=window, rot=rot,
+                         norm_over=norm_over, gate=True, v_mix=v_mix, mix_key=mix_key)
 
 
 class DifferentialAttention:

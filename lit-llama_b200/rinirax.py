@@ -164,7 +164,7 @@ class Rinirax:
             raise RuntimeError("32-bit products of this model (router, float32 mode) must be true f32: torch.backends.cuda.matmul.allow_tf32 is on")
         hist = self.depth.history(ctx, D, dev)                      # [layers + 1, T, D]: the embedding output, then every layer's own result
         x = hist[0]
-        S.check(lib.b2l_seq_embed(_p(tokens), int(tokens.dtype == torch.int64), _p(self.embed), ctx.act, 1.0, _p(x), T, D, self.vocab, ctx.stream),
+        S.check(lib.b2l_seq_embed(_p(tokens), int(tokens.dtype == torch.int64), _p(self.embed), ctx.act, 1.0, _p(x), None, T, D, self.vocab, ctx.stream),
                 "b2l_seq_embed")
         n = T if want is None else int(want.numel())
         L = len(self.layers)

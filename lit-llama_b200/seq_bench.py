@@ -231,7 +231,7 @@ def kernel_table(model, engine, T: int, device, timer: _Timer, peaks: dict) -> L
         y = torch.randn(tt, D, device=device).to(dt)
         h = torch.empty(tt, D, dtype=dt, device=device)
         w = torch.ones(D, dtype=dt, device=device)
-        t = timer(lambda: S.check(lib.b2l_seq_norm_add_norm(M._p(y), M._p(w), 1e-6, M._p(x), M._p(w), M._p(h), tt, D, ctx.act, ctx.stream), "k"))
+        t = timer(lambda: S.check(lib.b2l_seq_norm_add_norm(M._p(y), M._p(w), 1e-6, 1.0, M._p(x), M._p(w), M._p(h), tt, D, ctx.act, ctx.stream), "k"))
         add("seq_norm_add_norm_kernel", "rmsnorm_kernel + add_kernel", t, tt * D * (es + 4 + 4 + es))
         mlp = model.layers[0].mlp
         gu = torch.randn(tt, 2 * mlp.ff, device=device).to(dt)

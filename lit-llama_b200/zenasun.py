@@ -167,7 +167,7 @@ class Zenasun:
         if torch.backends.cuda.matmul.allow_tf32:
             raise RuntimeError("32-bit products of this model (router, float32 mode) must be true f32: torch.backends.cuda.matmul.allow_tf32 is on")
         x = torch.empty((T, D), dtype=torch.float32, device=dev)
-        S.check(lib.b2l_seq_embed(_p(tokens), int(tokens.dtype == torch.int64), _p(self.embed), ctx.act, self.config.embedding_scale, _p(x), T, D,
+        S.check(lib.b2l_seq_embed(_p(tokens), int(tokens.dtype == torch.int64), _p(self.embed), ctx.act, self.config.embedding_scale, _p(x), None, T, D,
                                   self.vocab, ctx.stream), "b2l_seq_embed")
         h1 = torch.empty((T, D), dtype=self.dtype, device=dev)
         h2 = torch.empty((T, D), dtype=self.dtype, device=dev)

@@ -97,14 +97,14 @@ def kernel_table(model, engine, T: int, device, timer, peaks: dict) -> List[dict
         add(f"seq_hc_step_kernel ({n_s} streams: write + read + norm)", tt, t, tt * D * (es + 8 * n_s + es))
         x1 = torch.randn(tt, D, device=device)
         h1 = torch.empty(tt, D, dtype=dt, device=device)
-        t = timer(lambda: S.check(lib.b2l_seq_norm_add_norm(M._p(y), M._p(w), eps, M._p(x1), M._p(w), M._p(h1), tt, D, ctx.act, ctx.stream), "k"))
+        t = timer(lambda: S.check(lib.b2l_seq_norm_add_norm(M._p(y), M._p(w), eps, 1.0, M._p(x1), M._p(w), M._p(h1), tt, D, ctx.act, ctx.stream), "k"))
         add("  like: seq_norm_add_norm_kernel (one stream: post-norm + add + norm)", tt, t, tt * D * (es + 4 + 4 + es))
         # ---- embedding: the token row plus the hashed pair row into every stream, against the plain embedding
         emb = model.embedding
         tk = torch.randint(0, emb.vocab, (tt,), device=device)
         t = timer(lambda: emb.forward(tk, ctx))
         add(f"seq_embed_pair_kernel (token + pair rows into {n_s} streams)", tt, t, tt * D * (2 * es + 4 * n_s))
-        t = timer(lambda: S.check(lib.b2l_seq_embed(M._p(tk), 1, M._p(emb.embed), ctx.act, 1.0, M._p(x1), tt, D, emb.vocab, ctx.stream), "k"))
+        t = timer(lambda: S.check(lib.b2l_seq_embed(M._p(tk), 1, M._p(emb.embed), ctx.act, 1.0, M._p(x1), None, tt, D, emb.vocab, ctx.stream), "k"))
         add("  like: seq_embed_kernel (token row into one stream)", tt, t, tt * D * (es + 4))
         # ---- attention operands
         proj = torch.randn(tt, att.w_in.shape[0], device=device).to(dt)

@@ -479,7 +479,7 @@ def test_post_norm_residual_pre_norm_all_widths(D, dtype):
     x, y, w1, w2 = torch.randn(T, D), (torch.randn(T, D) * 3).to(dtype), (torch.rand(D) + 0.5).to(dtype), (torch.rand(D) + 0.5).to(dtype)
     for nxt in (True, False):
         dx, h = dev(x.clone()), torch.zeros(T, D, device=DEV, dtype=dtype)
-        S.check(S.lib().b2l_seq_norm_add_norm(M._p(dev(y)), M._p(dev(w1)), 1e-5, M._p(dx), M._p(dev(w2)) if nxt else None, M._p(h) if nxt else None, T, D,
+        S.check(S.lib().b2l_seq_norm_add_norm(M._p(dev(y)), M._p(dev(w1)), 1e-5, 1.0, M._p(dx), M._p(dev(w2)) if nxt else None, M._p(h) if nxt else None, T, D,
                                               ctx.act, ctx.stream), "nan")
         x2 = x.double() + O.rms_norm(y.double(), w1.double(), 1e-5)
         assert rel(dx, x2) < 1e-6
@@ -520,7 +520,7 @@ def test_row_kernels():
     ctx = _ctx(T)
     x, y, w1, w2 = torch.randn(T, D), torch.randn(T, D) * 3, torch.rand(D) + 0.5, torch.rand(D) + 0.5
     dx, h = x.to(DEV), torch.empty(T, D, device=DEV)
-    S.check(lib.b2l_seq_norm_add_norm(M._p(dev(y)), M._p(dev(w1)), 1e-5, M._p(dx), M._p(dev(w2)), M._p(h), T, D, ctx.act, ctx.stream), "nan")
+    S.check(lib.b2l_seq_norm_add_norm(M._p(dev(y)), M._p(dev(w1)), 1e-5, 1.0, M._p(dx), M._p(dev(w2)), M._p(h), T, D, ctx.act, ctx.stream), "nan")
     x2 = x.double() + O.rms_norm(y.double(), w1.double(), 1e-5)
     assert rel(dx, x2) < 1e-6 and rel(h, O.rms_norm(x2, w2.double(), 1e-5)) < 1e-6
     rows = torch.tensor([4, 0, 4], dtype=torch.int32, device=DEV)
@@ -533,7 +533,7 @@ def test_row_kernels():
     assert rel(mid, O.gelu_tanh(gu[:, :33].double()) * gu[:, 33:].double()) < 1e-6
     tab, tok = torch.randn(11, D), torch.tensor([3, 10, 0, 3, 7, 1])
     emb = torch.empty(T, D, device=DEV)
-    S.check(lib.b2l_seq_embed(M._p(dev(tok)), 1, M._p(dev(tab)), ctx.act, 2.5, M._p(emb), T, D, 11, ctx.stream), "embed")
+    S.check(lib.b2l_seq_embed(M._p(dev(tok)), 1, M._p(dev(tab)), ctx.act, 2.5, M._p(emb), None, T, D, 11, ctx.stream), "embed")
     assert torch.equal(emb.cpu(), tab[tok] * 2.5)
     n, group = 48, 12
     o, gate, wn = torch.randn(T, n), torch.randn(T, n), torch.rand(n) + 0.5
