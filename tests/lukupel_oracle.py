@@ -87,12 +87,15 @@ def log_gates(h, W, p, cap):
     return i, -torch.log1p(torch.exp(-z))
 
 
-def matrix_memory(q, k, v, log_i, log_f):
-    """One head, token by token: q, k [T, K] (q already scaled), v [T, V], the two log gates [T] -> read-outs [T, V]."""
+def matrix_memory(q, k, v, log_i, log_f, lose=None):
+    """One head, token by token: q, k [T, K] (q already scaled), v [T, V], the two log gates [T] -> read-outs [T, V].
+    lose = (token, "S" | "n" | "m"): a planted mistake, that part of the state is gone before the token."""
     T, K, V = q.shape[0], q.shape[1], v.shape[1]
     S, n, m = torch.zeros(K, V, dtype=F64), torch.zeros(K, dtype=F64), 0.0
     out = torch.zeros(T, V, dtype=F64)
     for t in range(T):
+        if lose and lose[0] == t:
+            S, n, m = S * (lose[1] != "S"), n * (lose[1] != "n"), m * (lose[1] != "m")
         i, f = float(log_i[t]), float(log_f[t])
         new = max(f + m, i)
         keep, put = math.exp(f + m - new), math.exp(i - new)
@@ -103,13 +106,13 @@ def matrix_memory(q, k, v, log_i, log_f):
     return out
 
 
-def mlstm(h, W, p, c, eps):
+def mlstm(h, W, p, c, eps, lose=None):
     T, H, K, V = h.shape[0], c["heads"], c["dim"], c["vdim"]
     q = (h @ w64(W, p + "q").T).view(T, H, K) * K ** -0.5
     k = (h @ w64(W, p + "k").T).view(T, H, K)
     v = (h @ w64(W, p + "v").T).view(T, H, V)
     log_i, log_f = log_gates(h, W, p, c["gate_cap"])
-    o = torch.stack([matrix_memory(q[:, a], k[:, a], v[:, a], log_i[:, a], log_f[:, a]) for a in range(H)], dim=1)
+    o = torch.stack([matrix_memory(q[:, a], k[:, a], v[:, a], log_i[:, a], log_f[:, a], lose) for a in range(H)], dim=1)
     o = unit_rms(o, eps).reshape(T, H * V) * w64(W, p + "norm") * torch.sigmoid(h @ w64(W, p + "g").T)
     return o @ w64(W, p + "o").T
 
