@@ -134,7 +134,7 @@ __global__ void __launch_bounds__(128) seq_mlstm_readout_kernel(b2l_seq_mlstm_ar
 }
 
 // ---- a single token: cluster = one head, CTA rank r = value columns [r * per, (r + 1) * per).
-constexpr int STEP_THREADS = 256, STEP_CLUSTER = 8;
+constexpr int STEP_THREADS = 512, STEP_CLUSTER = 8, STEP_U = 4;      // STEP_THREADS: the most a CTA gets
 
 __device__ __forceinline__ void cluster_arrive() { asm volatile("barrier.cluster.arrive.release;" ::: "memory"); }
 __device__ __forceinline__ void cluster_wait() { asm volatile("barrier.cluster.wait.acquire;" ::: "memory"); }
@@ -149,7 +149,7 @@ template <typename act_t, bool VEC>
 __global__ void __launch_bounds__(STEP_THREADS) seq_mlstm_step_kernel(b2l_seq_mlstm_args a, int per, int G) {
   extern __shared__ __align__(16) float smem[];
   __shared__ float red[32], part[STEP_CLUSTER];
-  const int rank = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int rank = blockIdx.x, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, threads = blockDim.x;
   const int K = a.K, V = a.V, Kp = (K + 3) & ~3, slot = a.meta[0];
   float* sq = smem;                                    // [Kp] q times q_mult
   float* sk = sq + Kp;                                 // [Kp] put * k
@@ -163,7 +163,7 @@ __global__ void __launch_bounds__(STEP_THREADS) seq_mlstm_step_kernel(b2l_seq_ml
 
   float* pn = a.state_n + ((size_t)slot * a.heads + h) * K;
   float nq = 0.f;
-  for (int i = tid; i < Kp; i += STEP_THREADS) {
+  for (int i = tid; i < Kp; i += threads) {
     const float q = i < K ? row[a.q_off + (size_t)h * K + i] * a.q_mult : 0.f;
     const float k = i < K ? put * row[a.k_off + (size_t)h * K + i] : 0.f;
     sq[i] = q;
@@ -176,43 +176,65 @@ __global__ void __launch_bounds__(STEP_THREADS) seq_mlstm_step_kernel(b2l_seq_ml
   const int c0 = rank * per, nc = max(0, min(per, V - c0));
   float* S = a.state_S + (((size_t)slot * a.heads + h) * V + c0) * K;
   const float* v = row + a.v_off + (size_t)h * V + c0;
-  const int cpw = 32 / G, sub = lane / G, r = lane - sub * G;
-  for (int cb = warp * cpw; cb < nc; cb += (STEP_THREADS / 32) * cpw) {
-    const int c = cb + sub;
-    float dot = 0.f;
-    if (c < nc) {
-      const float vc = v[c];
-      float* Sc = S + (size_t)c * K;
-      if (VEC) {
-        for (int i = r * 4; i < K; i += G * 4) {
-          float4 s = *reinterpret_cast<float4*>(Sc + i);
-          const float4 k4 = *reinterpret_cast<const float4*>(sk + i), q4 = *reinterpret_cast<const float4*>(sq + i);
-          s.x = fmaf(keep, s.x, k4.x * vc); s.y = fmaf(keep, s.y, k4.y * vc);
-          s.z = fmaf(keep, s.z, k4.z * vc); s.w = fmaf(keep, s.w, k4.w * vc);
-          *reinterpret_cast<float4*>(Sc + i) = s;
-          dot = fmaf(s.x, q4.x, dot); dot = fmaf(s.y, q4.y, dot); dot = fmaf(s.z, q4.z, dot); dot = fmaf(s.w, q4.w, dot);
+  // A lane group owns column cb + sub; STEP_U columns, cpw * warps apart, are in flight at once.
+  const int cpw = 32 / G, sub = lane / G, r = lane - sub * G, stride = (threads >> 5) * cpw;
+  for (int cb = warp * cpw; cb < nc; cb += stride * STEP_U) {
+    float dot[STEP_U], vc[STEP_U];
+    float* Sc[STEP_U];
+    bool on[STEP_U];
+#pragma unroll
+    for (int u = 0; u < STEP_U; ++u) {
+      const int c = cb + sub + u * stride;
+      on[u] = c < nc;
+      vc[u] = on[u] ? v[c] : 0.f;
+      Sc[u] = S + (size_t)(on[u] ? c : 0) * K;
+      dot[u] = 0.f;
+    }
+    if (VEC) {
+      for (int i = r * 4; i < K; i += G * 4) {
+        const float4 k4 = *reinterpret_cast<const float4*>(sk + i), q4 = *reinterpret_cast<const float4*>(sq + i);
+        float4 s[STEP_U];
+#pragma unroll
+        for (int u = 0; u < STEP_U; ++u) s[u] = on[u] ? *reinterpret_cast<const float4*>(Sc[u] + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int u = 0; u < STEP_U; ++u) {
+          s[u].x = fmaf(keep, s[u].x, k4.x * vc[u]); s[u].y = fmaf(keep, s[u].y, k4.y * vc[u]);
+          s[u].z = fmaf(keep, s[u].z, k4.z * vc[u]); s[u].w = fmaf(keep, s[u].w, k4.w * vc[u]);
+          if (on[u]) *reinterpret_cast<float4*>(Sc[u] + i) = s[u];
+          dot[u] = fmaf(s[u].x, q4.x, dot[u]); dot[u] = fmaf(s[u].y, q4.y, dot[u]);
+          dot[u] = fmaf(s[u].z, q4.z, dot[u]); dot[u] = fmaf(s[u].w, q4.w, dot[u]);
         }
-      } else {
-        for (int i = r; i < K; i += G) {
-          const float s = fmaf(keep, Sc[i], sk[i] * vc);
-          Sc[i] = s;
-          dot = fmaf(s, sq[i], dot);
+      }
+    } else {
+      for (int i = r; i < K; i += G) {
+#pragma unroll
+        for (int u = 0; u < STEP_U; ++u) {
+          if (on[u]) {
+            const float s = fmaf(keep, Sc[u][i], sk[i] * vc[u]);
+            Sc[u][i] = s;
+            dot[u] = fmaf(s, sq[i], dot[u]);
+          }
         }
       }
     }
-    for (int o = 1; o < G; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
-    if (r == 0 && c < nc) so[c] = dot * inv;
+    for (int o = 1; o < G; o <<= 1) {
+#pragma unroll
+      for (int u = 0; u < STEP_U; ++u) dot[u] += __shfl_xor_sync(0xffffffffu, dot[u], o);
+    }
+#pragma unroll
+    for (int u = 0; u < STEP_U; ++u)
+      if (r == 0 && on[u]) so[cb + sub + u * stride] = dot[u] * inv;
   }
   __syncthreads();
   float ss = 0.f;
-  for (int c = tid; c < nc; c += STEP_THREADS) ss += so[c] * so[c];
+  for (int c = tid; c < nc; c += threads) ss += so[c] * so[c];
   ss = block_sum(ss, red);
   cluster_wait();
   if (tid < (int)gridDim.x) store_to_rank(part + rank, tid, ss);
   cluster_arrive();
   cluster_wait();                                      // all sums have arrived; m and n have been read by every CTA
   if (rank == 0) {
-    for (int i = tid; i < K; i += STEP_THREADS) pn[i] = fmaf(keep, pn[i], sk[i]);
+    for (int i = tid; i < K; i += threads) pn[i] = fmaf(keep, pn[i], sk[i]);
     if (tid == 0) *pm = m;
   }
   ss = 0.f;
@@ -220,16 +242,16 @@ __global__ void __launch_bounds__(STEP_THREADS) seq_mlstm_step_kernel(b2l_seq_ml
   const float rr = 1.f / sqrtf(ss / (float)V + a.eps);
   const float* g = row + a.g_off + (size_t)h * V + c0;
   const act_t* w = (const act_t*)a.w_norm + (size_t)h * V + c0;
-  for (int c = tid; c < nc; c += STEP_THREADS) st_act((act_t*)a.out, (size_t)h * V + c0 + c, so[c] * rr * ld_act(w, c) * sigmoid_f(g[c]));
+  for (int c = tid; c < nc; c += threads) st_act((act_t*)a.out, (size_t)h * V + c0 + c, so[c] * rr * ld_act(w, c) * sigmoid_f(g[c]));
 }
 
 static DynSmemCache g_step_smem[4];
 
 template <typename act_t, bool VEC>
-static int launch_step(const b2l_seq_mlstm_args* a, int per, int C, int G, size_t smem, cudaStream_t s, DynSmemCache& cache) {
+static int launch_step(const b2l_seq_mlstm_args* a, int per, int C, int G, int threads, size_t smem, cudaStream_t s, DynSmemCache& cache) {
   int rc = ensure_dyn_smem(seq_mlstm_step_kernel<act_t, VEC>, smem, cache);
   if (rc) return rc;
-  LaunchCfg cfg(dim3((unsigned)C, (unsigned)a->heads), dim3(STEP_THREADS), smem, s, false, C);
+  LaunchCfg cfg(dim3((unsigned)C, (unsigned)a->heads), dim3((unsigned)threads), smem, s, false, C);
   B2L_CUDA(cudaLaunchKernelEx(&cfg.cfg, seq_mlstm_step_kernel<act_t, VEC>, *a, per, G));
   return 0;
 }
@@ -284,13 +306,15 @@ extern "C" int b2l_seq_mlstm_step(const b2l_seq_mlstm_args* a, b2l_stream_t stre
   const int want = vec ? (a->K + 3) / 4 : a->K;
   int G = 1;
   while (G < 32 && G < want) G <<= 1;
+  // a warp takes STEP_U rounds of 32 / G columns at once
+  const int threads = per * G > 32 * STEP_U * 8 ? STEP_THREADS : STEP_THREADS / 2;
   const size_t smem = sizeof(float) * (2 * (size_t)((a->K + 3) & ~3) + per);
   B2L_CHECK_SUPPORTED(smem <= 200 * 1024, "b2l_seq_mlstm_step: head of %d x %d too large", a->K, a->V);
   cudaStream_t s = (cudaStream_t)stream;
   if (a->act_dtype == B2L_BF16) {
-    rc = vec ? launch_step<__nv_bfloat16, true>(a, per, C, G, smem, s, g_step_smem[0]) : launch_step<__nv_bfloat16, false>(a, per, C, G, smem, s, g_step_smem[1]);
+    rc = vec ? launch_step<__nv_bfloat16, true>(a, per, C, G, threads, smem, s, g_step_smem[0]) : launch_step<__nv_bfloat16, false>(a, per, C, G, threads, smem, s, g_step_smem[1]);
   } else if (a->act_dtype == B2L_F32) {
-    rc = vec ? launch_step<float, true>(a, per, C, G, smem, s, g_step_smem[2]) : launch_step<float, false>(a, per, C, G, smem, s, g_step_smem[3]);
+    rc = vec ? launch_step<float, true>(a, per, C, G, threads, smem, s, g_step_smem[2]) : launch_step<float, false>(a, per, C, G, threads, smem, s, g_step_smem[3]);
   } else {
     set_error("b2l_seq_mlstm_step: act_dtype %d unsupported", a->act_dtype);
     return B2L_E_UNSUPPORTED;
