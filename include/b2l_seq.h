@@ -243,7 +243,7 @@ int b2l_seq_latent_prep(const float* proj, int ld, int q_off, int q_rank, const 
 /* Causal softmax attention with a learned sink per head over keys 0 .. pos0 + t, or, with window > 0, over the keys
  * pos0 + t - window + 1 .. pos0 + t (the query's own position and the window - 1 before it):
  *   weights exp(score_j) / (exp(sink[h]) + sum_j exp(score_j)),  score = (q . key_j[score_off:]) * scale
- *   (sink null: ordinary softmax, no sink term)
+ *   (sink null: ordinary softmax, no sink term), times the gate when one is given
  *   out[t, h*vdim : (h+1)*vdim] = sum_j weight_j key_j[0 : vdim]
  * A key row is [A (n_a entries) | B (n_b entries)]: A belongs to a key group (row j at key_a + slot*slot_stride_a +
  * group*hska + j*ldka), B is shared by all groups (key_b + slot*slot_stride_b + j*ldkb); heads_per_group consecutive
@@ -268,8 +268,40 @@ typedef struct {
   float scale;
   int T, heads, heads_per_group, n_a, n_b, vdim, score_off, splits, act_dtype;
   int window;                      /* 0: every earlier position; > 0: a sliding window of that many positions */
+  const float* gate; int ldg;      /* f32 [T, ldg] or null: out[t, h*vdim + v] is multiplied by sigmoid(gate[t, h*vdim + v]) */
+  int partial;                     /* stop at the work space (also with one split): b2l_seq_latent_up merges it; out is not written */
 } b2l_seq_latent_attn_args;
 int b2l_seq_latent_attention(const b2l_seq_latent_attn_args* a, b2l_stream_t stream);
+
+/* Operands of latent attention whose queries are a direct image of the layer's input, from one f32 product proj [T, ld] with
+ * q at q_off (heads x [dn unrotated | dr rotated]) and [c' | k_r] (rank + dr) at kv_off:
+ *   cache[slot][pos0 + t] = [ rmsnorm(c') * w_kv | rotate(k_r) ]     as b2l_seq_latent_prep
+ *   and the queries, rotated parts turned by position, in one of three forms:
+ *     q_full  f32 [T][heads*(dn + dr)]                                     for the expanded form
+ *     q_nope  act [heads][T][dn]      and q_rot f32 [T][heads][dr]         for the latent form, W_uk still to be applied
+ *     q_lat   f32 [heads][T][rank]    and q_rot                            for the latent form: q_lat = W_uk,h^T q_h is computed in
+ *                                                                          the same launch (w_uk act [heads][dn][rank]; a few tokens) */
+typedef struct {
+  const float* proj; int ld, q_off, kv_off;
+  int heads, dn, dr, rank;
+  const void* w_kv;
+  const float* freq; int rot_dims, interleaved; float rot_mult, eps;
+  const int* meta; void* cache; int max_pos;
+  float* q_full; void* q_nope; float* q_rot;
+  const void* w_uk; float* q_lat;
+  int T, act_dtype;
+} b2l_seq_latent_operands_args;
+int b2l_seq_latent_operands(const b2l_seq_latent_operands_args* a, b2l_stream_t stream);
+
+/* The latent form's tail for a few tokens: merges the key splits of `partial` attention results (work f32
+ * [splits][T*heads][rank + 2]) with the sink, applies the value up-projection (w_uv act [heads*vdim][rank]) to the f32 row
+ * and the gate: out[t, h*vdim + j] = (w_uv[h*vdim + j] . o_lat[t, h]) * sigmoid(gate[t, h*vdim + j])      (gate f32 or null) */
+int b2l_seq_latent_up(const float* work, const float* sink, const void* w_uv, const float* gate, int ldg, void* out, int ldo, int T, int heads,
+                      int rank, int vdim, int splits, int act_dtype, b2l_stream_t stream);
+
+/* out[t, h*V + c] = in[t*ld_t + h*ld_h + c] * sigmoid(gate[t*ldg + h*V + c]): heads of any layout, gated (gate f32, null: copied). */
+int b2l_seq_head_gate(const void* in, long long ld_t, long long ld_h, const float* gate, int ldg, void* out, int ldo, int T, int heads, int V,
+                      int act_dtype, b2l_stream_t stream);
 int b2l_seq_latent_attention_warps(int T, int heads_per_group);    /* warps per CTA that own rows: 4 rows per warp */
 
 /* ---- mixture of experts ----
@@ -278,8 +310,10 @@ int b2l_seq_latent_attention_warps(int T, int heads_per_group);    /* warps per 
  * neighbours, a group's score is the sum of its `group_top` largest choice scores (1: its largest), only experts of the
  * `keep` best groups can be chosen (ties to the lower group);
  * idx[t, :] = the `top` largest choice scores among them (best first, ties to the lower index);
- * weights[t, k] = weight_scale * s[idx] / (sum of the chosen s + 1e-20) when `renormalize`, else weight_scale * s[idx]. */
-enum { B2L_SEQ_SCORE_SOFTMAX = 0, B2L_SEQ_SCORE_SIGMOID = 1 };
+ * weights[t, k] = weight_scale * s[idx] / (sum of the chosen s + 1e-20) when `renormalize`, else weight_scale * s[idx].
+ * B2L_SEQ_SCORE_CHOSEN_SOFTMAX (renormalize set): `correction` is a bias of the logits; choice = logits + correction, and the
+ * weights are the softmax of those over the chosen experts alone. */
+enum { B2L_SEQ_SCORE_SOFTMAX = 0, B2L_SEQ_SCORE_SIGMOID = 1, B2L_SEQ_SCORE_CHOSEN_SOFTMAX = 2 };
 int b2l_seq_moe_route(const float* logits, int ld, const float* correction, int n, int groups, int keep, int top, int score_fn,
                       int renormalize, int group_top, float weight_scale, int* idx, float* weights, int T, b2l_stream_t stream);
 
@@ -292,10 +326,13 @@ int b2l_seq_moe_route_fused(const void* h, int ldh, const void* w_router, const 
  * with w_gate_up act [n_real][2*ff][D] (gate rows, then up rows), w_down act [n_real][D][ff] and the gated unit of
  * b2l_seq_gated_act (`act`, `limit`); e >= n_real: h itself.
  * y[t] = sum_k weights[t, k] * expert_idx[t,k](h[t]), or, with weight_input, sum_k expert_idx[t,k](weights[t, k] * h[t])
- * (the weighted input passes through the storage type).  mid: act [T*top, ff] scratch. */
+ * (the weighted input passes through the storage type).  With ff_shared > 0 one more expert (w_shared_gate_up act
+ * [2*ff_shared][D], w_shared_down act [D][ff_shared]) runs on every h[t] in the same launches and is added unweighted.
+ * mid: act scratch of T*top*ff + T*ff_shared entries. */
 int b2l_seq_moe_experts_small(const void* h, int ldh, const void* w_gate_up, const void* w_down, const int* idx,
                               const float* weights, void* mid, void* y, int ldy, int T, int D, int ff, int n_real, int top,
-                              int act, float limit, int weight_input, int act_dtype, b2l_stream_t stream);
+                              int act, float limit, int weight_input, const void* w_shared_gate_up, const void* w_shared_down, int ff_shared,
+                              int act_dtype, b2l_stream_t stream);
 
 /* Long portions: the N = T*top assignments a = t*top + k sorted by expert.  offsets int32[n_real + 1]: expert e owns
  * the sorted places offsets[e] .. offsets[e+1]-1; perm[p] = assignment at place p; inv[a] = place of assignment a
@@ -305,9 +342,10 @@ int b2l_seq_moe_sort(const int* idx, int N, int n_real, int* offsets, int* curso
  * an expert's input) for p < *n_rows (device int32: offsets[n_real]); launched over N rows. */
 int b2l_seq_moe_gather(const void* h, int ldh, const int* perm, const int* n_rows, const float* row_scale, int top, void* xg, int N,
                        int D, int act_dtype, b2l_stream_t stream);
-/* y[t] = sum_k weights[t, k] * (inv[a] >= 0 ? yg[inv[a]] : h[t]); weights null: every weight is 1. */
-int b2l_seq_moe_combine(const void* yg, const int* inv, const float* weights, const void* h, int ldh, void* y, int ldy, int T,
-                        int D, int top, int act_dtype, b2l_stream_t stream);
+/* y[t] = sum_k weights[t, k] * (inv[a] >= 0 ? yg[inv[a]] : h[t]); weights null: every weight is 1.  add (act [T, ldadd],
+ * may be null): one more summand, e.g. the output of an expert that every token uses. */
+int b2l_seq_moe_combine(const void* yg, const int* inv, const float* weights, const void* h, int ldh, const void* add, int ldadd,
+                        void* y, int ldy, int T, int D, int top, int act_dtype, b2l_stream_t stream);
 
 /* ---- several residual streams, token-pair embedding, attention operands ----
  * Token embedding plus a hashed token-pair embedding, written into `streams` equal residual streams x [T][streams][D]:
@@ -350,6 +388,27 @@ int b2l_seq_depth_step(const void* y1, const void* y2, const float* x_in, float*
                        const void* w_next, const void* b_next, int norm_kind, float eps, void* h, int T, int D, int act_dtype,
                        b2l_stream_t stream);
 
+/* The plain residual step, one row per token (x f32 [T, D]):
+ *   x_out = x_in + base + vec + (y1 + y2)     base f32 [T, D], vec act [D] (the same for every token), y1, y2 act [T, D]; each may be null
+ *   h     = norm(x_out) as b2l_seq_norm       act [T, D]; w, b and h may be null
+ *   split = [hi | lo] of x_out                act [T, 2 D], may be null: hi = x_out in the storage type, lo = what that rounding
+ *                                             lost, so that [hi | lo] [W | W]^T is the product of W with the f32 row
+ * x_out may be x_in, or null when the row itself is not needed (not for rows wider than 4096 entries, 8192 when D is a
+ * multiple of 4 and everything is 16-byte aligned). */
+typedef struct {
+  const float* x_in; const float* base; const void* vec; const void* y1; const void* y2;
+  float* x_out; void* split;
+  const void* w; const void* b; void* h;
+  float eps; int norm_kind;
+  int T, D, act_dtype;
+} b2l_seq_residual_args;
+int b2l_seq_residual_step(const b2l_seq_residual_args* a, b2l_stream_t stream);
+
+/* A product with f32 rows for a few tokens, f32 throughout: out[t, i] = W[i, :] . x[t, :] + base[t, i] + vec[i]
+ * (W act [N, K], x f32 [T, K], base f32 [T, N] or null, vec act [N] or null, out f32 [T, N], not x). */
+int b2l_seq_linear_few(const void* w, const float* x, const float* base, const void* vec, float* out, int T, int N, int K, int act_dtype,
+                       b2l_stream_t stream);
+
 /* z <- z * mult in place on f32 (a constant scale of the logits). */
 int b2l_seq_scale(float* z, size_t n, float mult, b2l_stream_t stream);
 
@@ -371,6 +430,7 @@ typedef struct {
   int T, heads, kv_heads, K, V, act_dtype;
   int unit_rms;                   /* null norm weights: every head of q and k, after its rotation, divided by its root mean
                                      square (eps) over K */
+  float temp_coef; int temp_every;    /* temp_every > 0: q_out at position p times 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) */
 } b2l_seq_qkv_prep_args;
 int b2l_seq_qkv_prep(const b2l_seq_qkv_prep_args* a, b2l_stream_t stream);
 

@@ -18,6 +18,7 @@ from .zenasun import Zenasun, ZenasunConfig
 from .zuvevik import Zuvevik, ZuvevikConfig
 from .rinirax import Rinirax, RiniraxConfig
 from .lukupel import Lukupel, LukupelConfig
+from .malulorn import Malulorn, MalulornConfig
 from .state import SequenceStatePool, StateSpec
 from .engine import Engine
 from .registry import load_model, register
@@ -26,5 +27,6 @@ __all__ = [
     "LLaMA", "LLaMAConfig", "Block", "CausalSelfAttention", "MLP", "RMSNorm", "build_rope_cache", "apply_rope",
     "ColBlockQuantizedLinear", "Linear8bitLt", "find_multiple", "llama_model_lookup", "generate", "sample_probs", "sample_token", "patch_reference", "TPLLaMA", "shard_state_dict",
     "Lugovik", "LugovikConfig", "Zenasun", "ZenasunConfig", "Zuvevik", "ZuvevikConfig", "Rinirax", "RiniraxConfig", "Lukupel", "LukupelConfig",
+    "Malulorn", "MalulornConfig",
     "SequenceStatePool", "StateSpec", "Engine", "load_model", "register",
 ]

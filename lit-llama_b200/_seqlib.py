@@ -10,7 +10,7 @@ from . import _build
 B2L_BF16, B2L_F32 = 0, 1
 ACT_GELU_TANH, ACT_SILU, ACT_SIGMOID, ACT_CLAMPED_SWISH, ACT_XIELU, ACT_NONE, ACT_RELU2 = 0, 1, 2, 3, 4, 5, 6
 NORM_RMS, NORM_LAYER = 0, 1
-SCORE_SOFTMAX, SCORE_SIGMOID = 0, 1
+SCORE_SOFTMAX, SCORE_SIGMOID, SCORE_CHOSEN_SOFTMAX = 0, 1, 2
 DECAY_EXP_SOFTPLUS, DECAY_SIGMOID_ROOT = 0, 1
 
 c_void_p, c_int, c_float, c_size_t = C.c_void_p, C.c_int, C.c_float, C.c_size_t
@@ -68,6 +68,31 @@ class LatentAttnArgs(C.Structure):
         ("T", c_int), ("heads", c_int), ("heads_per_group", c_int), ("n_a", c_int), ("n_b", c_int), ("vdim", c_int), ("score_off", c_int),
         ("splits", c_int), ("act_dtype", c_int),
         ("window", c_int),
+        ("gate", c_void_p), ("ldg", c_int),
+        ("partial", c_int),
+    ]
+
+
+class LatentOperandsArgs(C.Structure):
+    _fields_ = [
+        ("proj", c_void_p), ("ld", c_int), ("q_off", c_int), ("kv_off", c_int),
+        ("heads", c_int), ("dn", c_int), ("dr", c_int), ("rank", c_int),
+        ("w_kv", c_void_p),
+        ("freq", c_void_p), ("rot_dims", c_int), ("interleaved", c_int), ("rot_mult", c_float), ("eps", c_float),
+        ("meta", c_void_p), ("cache", c_void_p), ("max_pos", c_int),
+        ("q_full", c_void_p), ("q_nope", c_void_p), ("q_rot", c_void_p),
+        ("w_uk", c_void_p), ("q_lat", c_void_p),
+        ("T", c_int), ("act_dtype", c_int),
+    ]
+
+
+class ResidualArgs(C.Structure):
+    _fields_ = [
+        ("x_in", c_void_p), ("base", c_void_p), ("vec", c_void_p), ("y1", c_void_p), ("y2", c_void_p),
+        ("x_out", c_void_p), ("split", c_void_p),
+        ("w", c_void_p), ("b", c_void_p), ("h", c_void_p),
+        ("eps", c_float), ("norm_kind", c_int),
+        ("T", c_int), ("D", c_int), ("act_dtype", c_int),
     ]
 
 
@@ -93,6 +118,7 @@ class QkvPrepArgs(C.Structure):
         ("v_first", c_void_p), ("ldvf", c_int), ("lambda_", c_void_p), ("v_out", c_void_p),
         ("T", c_int), ("heads", c_int), ("kv_heads", c_int), ("K", c_int), ("V", c_int), ("act_dtype", c_int),
         ("unit_rms", c_int),
+        ("temp_coef", c_float), ("temp_every", c_int),
     ]
 
 
@@ -146,10 +172,10 @@ _SIGS = {
     "b2l_seq_moe_route_fused": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                                         c_void_p, c_void_p, c_int, c_int, c_void_p]),
     "b2l_seq_moe_experts_small": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                          c_int, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p]),
+                                          c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p]),
     "b2l_seq_moe_sort": (c_int, [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p]),
     "b2l_seq_moe_gather": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p]),
-    "b2l_seq_moe_combine": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b2l_seq_moe_combine": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "b2l_seq_embed_pair": (c_int, [c_void_p, c_int, c_void_p, c_void_p, c_float, c_void_p, c_void_p, C.c_longlong, C.c_longlong, c_int, c_void_p,
                                    c_int, c_int, c_int, c_int, c_int, c_void_p]),
     "b2l_seq_hc_step": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int,
@@ -166,6 +192,11 @@ _SIGS = {
     "b2l_seq_norm": (c_int, [c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]),
     "b2l_seq_depth_step": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float,
                                    c_void_p, c_int, c_int, c_int, c_void_p]),
+    "b2l_seq_latent_operands": (c_int, [C.POINTER(LatentOperandsArgs), c_void_p]),
+    "b2l_seq_latent_up": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b2l_seq_head_gate": (c_int, [c_void_p, C.c_longlong, C.c_longlong, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p]),
+    "b2l_seq_residual_step": (c_int, [C.POINTER(ResidualArgs), c_void_p]),
+    "b2l_seq_linear_few": (c_int, [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]),
     "b2l_seq_mlstm_step": (c_int, [C.POINTER(MlstmArgs), c_void_p]),
     "b2l_seq_mlstm_gates": (c_int, [C.POINTER(MlstmArgs), c_void_p]),
     "b2l_seq_mlstm_readout": (c_int, [C.POINTER(MlstmArgs), c_void_p]),

@@ -30,6 +30,36 @@ __device__ __forceinline__ float gated_pair(float a, float b, int act, float lim
   return (act == B2L_SEQ_ACT_GELU_TANH ? gelu_tanh_f(a) : (act == B2L_SEQ_ACT_SILU ? silu_f(a) : sigmoid_f(a))) * b;
 }
 
+// Dot product of a weight row with a vector in shared memory (f32); the warp's lanes stride the row.
+template <typename act_t>
+__device__ __forceinline__ float row_dot(const act_t* __restrict__ w, const float* __restrict__ x, int n, int lane, bool vec) {
+  float acc = 0.f;
+  if (vec) {                                         // 16-byte loads: n a multiple of 8 (bf16) / 4 (f32), aligned rows
+    constexpr int PER = 16 / sizeof(act_t);
+    for (int i = lane * PER; i < n; i += 32 * PER) {
+      const uint4 u = *reinterpret_cast<const uint4*>(w + i);
+      if (sizeof(act_t) == 2) {
+        const uint32_t ww[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+        for (int q = 0; q < 4; ++q) {
+          acc = fmaf(__uint_as_float(ww[q] << 16), x[i + 2 * q], acc);
+          acc = fmaf(__uint_as_float(ww[q] & 0xffff0000u), x[i + 2 * q + 1], acc);
+        }
+      } else {
+        acc = fmaf(__uint_as_float(u.x), x[i], acc);
+        acc = fmaf(__uint_as_float(u.y), x[i + 1], acc);
+        acc = fmaf(__uint_as_float(u.z), x[i + 2], acc);
+        acc = fmaf(__uint_as_float(u.w), x[i + 3], acc);
+      }
+    }
+  } else {
+    for (int i = lane; i < n; i += 32) acc = fmaf(ld_act(w, i), x[i], acc);
+  }
+  return warp_sum(acc);
+}
+
+static inline bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
+
 // Calls `fn.template operator()<T>()` with the element type of act_dtype.
 #define B2L_SEQ_DISPATCH(act_dtype, ...)                                   \
   do {                                                                     \

@@ -89,6 +89,114 @@ __global__ void __launch_bounds__(128) seq_latent_prep_kernel(const float* __res
   for (int i = rot_dims + threadIdx.x; i < rot_dim; i += blockDim.x) st_act(dst, rank + i, b[i]);
 }
 
+// Attention operands of one token when the queries are a direct image of the layer's input (no query latent), from the f32
+// product [.. q .. | c' | k_r ..]:
+//   blockIdx.y == 0: the cache row, as in the kernel above;
+//   blockIdx.y >= 1, q_lat null: all heads' queries by one CTA, either q_full (f32, [unrotated | rotated] per head) or q_nope
+//       (act, [heads][T][dn]) and q_rot (f32, [T][heads][dr]);
+//   blockIdx.y >= 1, q_lat given (a few tokens): head (y - 1) / chunks, LAT_ABS_COLS columns of q_lat = W_uk,h^T q_h, with the
+//       unrotated query in shared memory: a thread owns two columns and a quarter of the rows, the quarters are added at the
+//       end; the head's first chunk also writes q_rot.
+// Every CTA computes the angles it needs once per pair.
+constexpr int LAT_ABS_COLS = 128;
+
+template <typename act_t>
+__global__ void __launch_bounds__(256) seq_latent_operands_kernel(b2l_seq_latent_operands_args a, int chunks) {
+  extern __shared__ __align__(16) float op_smem[];                // cos | sin per pair, then (absorbed) q [dn]
+  __shared__ float red[32];
+  __shared__ float part[4][LAT_ABS_COLS];
+  const int t = blockIdx.x, tid = threadIdx.x, half = a.rot_dims / 2, dq = a.dn + a.dr;
+  const float* row = a.proj + (size_t)t * a.ld;
+  const int slot = a.meta[0], pos = a.meta[1] + t;
+  float* cs = op_smem;
+  float* sn = cs + half;
+  const int b = (int)blockIdx.y - 1;
+  const int h0 = a.q_lat ? b / chunks : 0, chunk = a.q_lat ? b - h0 * chunks : 0;
+  if (b < 0 || chunk == 0) {
+    for (int i = tid; i < half; i += blockDim.x) {
+      float s, c;
+      sincosf((float)pos * a.freq[i], &s, &c);
+      cs[i] = c * a.rot_mult;
+      sn[i] = s * a.rot_mult;
+    }
+  }
+  if (b < 0) {
+    const float* kv = row + a.kv_off;
+    float ss = 0.f;
+    for (int i = tid; i < a.rank; i += blockDim.x) ss += kv[i] * kv[i];
+    ss = block_sum(ss, red);                                      // also orders the angles before their use
+    __syncthreads();
+    if (pos < 0 || pos >= a.max_pos) return;                      // the pool never hands out such a position
+    const float r = 1.0f / sqrtf(ss / (float)a.rank + a.eps);
+    act_t* dst = (act_t*)a.cache + ((size_t)slot * a.max_pos + pos) * (size_t)(a.rank + a.dr);
+    for (int i = tid; i < a.rank; i += blockDim.x) st_act(dst, i, kv[i] * r * ld_act((const act_t*)a.w_kv, i));
+    const float* kr = kv + a.rank;
+    for (int i = tid; i < half; i += blockDim.x) {
+      const int iu = a.interleaved ? 2 * i : i, iv = a.interleaved ? 2 * i + 1 : i + half;
+      st_act(dst, a.rank + iu, kr[iu] * cs[i] - kr[iv] * sn[i]);
+      st_act(dst, a.rank + iv, kr[iv] * cs[i] + kr[iu] * sn[i]);
+    }
+    for (int i = a.rot_dims + tid; i < a.dr; i += blockDim.x) st_act(dst, a.rank + i, kr[i]);
+    return;
+  }
+  const float* q = row + a.q_off;
+  float* sq = sn + half;
+  if (a.q_lat)
+    for (int i = tid; i < a.dn; i += blockDim.x) sq[i] = q[(size_t)h0 * dq + i];
+  __syncthreads();
+  // rotated parts of the heads [h0, h1)
+  if (chunk == 0) {
+    const int h1 = a.q_lat ? h0 + 1 : a.heads, rest = a.dr - a.rot_dims, per = half + rest;
+    for (int i = tid; i < (h1 - h0) * per; i += blockDim.x) {
+      const int hd = h0 + i / per, j = i % per;
+      const float* p = q + (size_t)hd * dq + a.dn;
+      float* o = a.q_full ? a.q_full + ((size_t)t * a.heads + hd) * dq + a.dn : a.q_rot + ((size_t)t * a.heads + hd) * a.dr;
+      if (j < half) {
+        const int iu = a.interleaved ? 2 * j : j, iv = a.interleaved ? 2 * j + 1 : j + half;
+        const float u = p[iu], v = p[iv];
+        o[iu] = u * cs[j] - v * sn[j];
+        o[iv] = v * cs[j] + u * sn[j];
+      } else {
+        o[a.rot_dims + j - half] = p[a.rot_dims + j - half];
+      }
+    }
+  }
+  if (a.q_lat == nullptr) {
+    for (int i = tid; i < a.heads * a.dn; i += blockDim.x) {
+      const int hd = i / a.dn, j = i - hd * a.dn;
+      const float v = q[(size_t)hd * dq + j];
+      if (a.q_full) a.q_full[((size_t)t * a.heads + hd) * dq + j] = v;
+      else st_act((act_t*)a.q_nope, ((size_t)hd * a.T + t) * a.dn + j, v);
+    }
+    return;
+  }
+  const act_t* w = (const act_t*)a.w_uk + (size_t)h0 * a.dn * a.rank;
+  const int g = tid >> 6, lc = (tid & 63) * 2, col = chunk * LAT_ABS_COLS + lc;
+  float acc0 = 0.f, acc1 = 0.f;
+  if (col < a.rank) {
+    const bool two = col + 1 < a.rank;
+    if (sizeof(act_t) == 2 && (a.rank & 1) == 0) {                 // a column pair is one aligned 4-byte word
+#pragma unroll 16
+      for (int d = g; d < a.dn; d += 4) {
+        const uint32_t u = *reinterpret_cast<const uint32_t*>(w + (size_t)d * a.rank + col);
+        acc0 = fmaf(__uint_as_float(u << 16), sq[d], acc0);
+        acc1 = fmaf(__uint_as_float(u & 0xffff0000u), sq[d], acc1);
+      }
+    } else {
+#pragma unroll 8
+      for (int d = g; d < a.dn; d += 4) {
+        acc0 = fmaf(ld_act(w, (size_t)d * a.rank + col), sq[d], acc0);
+        if (two) acc1 = fmaf(ld_act(w, (size_t)d * a.rank + col + 1), sq[d], acc1);
+      }
+    }
+  }
+  part[g][lc] = acc0;
+  part[g][lc + 1] = acc1;
+  __syncthreads();
+  for (int i = tid; i < LAT_ABS_COLS && chunk * LAT_ABS_COLS + i < a.rank; i += blockDim.x)
+    a.q_lat[((size_t)h0 * a.T + t) * a.rank + chunk * LAT_ABS_COLS + i] = (part[0][i] + part[1][i]) + (part[2][i] + part[3][i]);
+}
+
 constexpr int LAT_RW = 4;       // rows (query, head) per warp
 constexpr int LAT_BN = 32;      // keys per tile: one per lane
 constexpr int LAT_LDK = 33;     // padded key count of the transposed tile
@@ -270,7 +378,7 @@ __global__ void __launch_bounds__(LAT_THREADS, VI <= 4 ? 3 : 1) seq_latent_atten
     const int row = row0 + warp * LAT_RW + r;
     if (row >= R) continue;
     const int t = row / hpg, h = group * hpg + row % hpg;
-    if (gridDim.y == 1) {
+    if (gridDim.y == 1 && !a.partial) {
       const float sink = a.sink ? a.sink[h] : -INFINITY;            // without a sink every row sees its own key: m is finite
       const float M = fmaxf(m[r], sink);
       const float e = expf(m[r] - M);                               // m = -inf (no key): 0
@@ -279,7 +387,7 @@ __global__ void __launch_bounds__(LAT_THREADS, VI <= 4 ? 3 : 1) seq_latent_atten
 #pragma unroll
       for (int i = 0; i < VI; ++i) {
         const int v = lane + 32 * i;
-        if (v < a.vdim) st_act(o, v, acc[r][i] * inv);
+        if (v < a.vdim) st_act(o, v, acc[r][i] * inv * (a.gate ? sigmoid_f(a.gate[(size_t)t * a.ldg + (size_t)h * a.vdim + v]) : 1.f));
       }
     } else {
       float* w = a.work + ((size_t)blockIdx.y * a.T * a.heads + (size_t)t * a.heads + h) * (size_t)(a.vdim + 2);
@@ -296,17 +404,8 @@ __global__ void __launch_bounds__(LAT_THREADS, VI <= 4 ? 3 : 1) seq_latent_atten
   }
 }
 
-// Merges the key splits of a row and adds the sink.  One CTA per row (t, h): warp 0 turns every split's running
-// maximum and sum into one factor exp(m_s - M) / denominator, then the threads own value entries and add the
-// splits' accumulators with independent loads.
-template <typename act_t>
-__global__ void __launch_bounds__(256) seq_latent_combine_kernel(const float* __restrict__ work, const float* __restrict__ sink,
-                                                                 act_t* __restrict__ out, int ldo, int R, int heads, int vdim, int splits) {
-  extern __shared__ float comb_f[];                      // [splits]
-  const int row = blockIdx.x, t = row / heads, h = row % heads;
-  const size_t stride = (size_t)(vdim + 2);
-  const float* w0 = work + (size_t)row * stride;
-  const size_t sstep = (size_t)R * stride;
+// The factors exp(m_s - M) / denominator of a row's key splits into comb_f, by warp 0; ends with a barrier.
+__device__ __forceinline__ void split_factors(const float* __restrict__ w0, size_t sstep, const float* __restrict__ sink, int h, int splits, float* comb_f) {
   if (threadIdx.x < 32) {
     const int lane = threadIdx.x;
     const float sk = sink ? sink[h] : -INFINITY;
@@ -325,14 +424,66 @@ __global__ void __launch_bounds__(256) seq_latent_combine_kernel(const float* __
     for (int s = lane; s < splits; s += 32) comb_f[s] *= inv;
   }
   __syncthreads();
-  act_t* o = out + (size_t)t * ldo + (size_t)h * vdim;
-  for (int v = threadIdx.x; v < vdim; v += blockDim.x) {
-    float acc = 0.f;
+}
+
+// Entry v of the merged row: the splits' accumulators added with independent loads.
+__device__ __forceinline__ float merged_entry(const float* __restrict__ w0, size_t sstep, int splits, const float* comb_f, int v) {
+  float acc = 0.f;
 #pragma unroll 16
-    for (int s = 0; s < splits; ++s) {
-      acc = fmaf(w0[(size_t)s * sstep + 2 + v], comb_f[s], acc);            // an empty split wrote zeros and has factor 0
-    }
-    st_act(o, v, acc);
+  for (int s = 0; s < splits; ++s) acc = fmaf(w0[(size_t)s * sstep + 2 + v], comb_f[s], acc);      // an empty split wrote zeros and has factor 0
+  return acc;
+}
+
+// Merges the key splits of a row, adds the sink and applies the gate.  One CTA per row (t, h): warp 0 turns every split's
+// running maximum and sum into one factor, then the threads own value entries.
+template <typename act_t>
+__global__ void __launch_bounds__(256) seq_latent_combine_kernel(const float* __restrict__ work, const float* __restrict__ sink,
+                                                                 const float* __restrict__ gate, int ldg, act_t* __restrict__ out, int ldo,
+                                                                 int R, int heads, int vdim, int splits) {
+  extern __shared__ float comb_f[];                      // [splits]
+  const int row = blockIdx.x, t = row / heads, h = row % heads;
+  const size_t stride = (size_t)(vdim + 2), sstep = (size_t)R * stride;
+  const float* w0 = work + (size_t)row * stride;
+  split_factors(w0, sstep, sink, h, splits, comb_f);
+  act_t* o = out + (size_t)t * ldo + (size_t)h * vdim;
+  for (int v = threadIdx.x; v < vdim; v += blockDim.x)
+    st_act(o, v, merged_entry(w0, sstep, splits, comb_f, v) * (gate ? sigmoid_f(gate[(size_t)t * ldg + (size_t)h * vdim + v]) : 1.f));
+}
+
+// A few tokens in the latent form: merge of the key splits, value up-projection and gate in one launch.  grid (T * heads,
+// chunks of LAT_UP_ROWS value entries): every CTA merges the whole latent row (f32, shared memory; the partials are in L2),
+// then a warp per value entry takes its dot product with the row of W_uv.
+constexpr int LAT_UP_ROWS = 32;
+
+template <typename act_t>
+__global__ void __launch_bounds__(256) seq_latent_up_kernel(const float* __restrict__ work, const float* __restrict__ sink, const act_t* __restrict__ w_uv,
+                                                            const float* __restrict__ gate, int ldg, act_t* __restrict__ out, int ldo, int R, int heads,
+                                                            int rank, int vdim, int splits, int vec) {
+  extern __shared__ float up_smem[];                     // merged latent [rank], factors [splits]
+  float* o_lat = up_smem;
+  float* comb_f = up_smem + rank;
+  const int row = blockIdx.x, t = row / heads, h = row % heads, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const size_t stride = (size_t)(rank + 2), sstep = (size_t)R * stride;
+  const float* w0 = work + (size_t)row * stride;
+  split_factors(w0, sstep, sink, h, splits, comb_f);
+  for (int v = threadIdx.x; v < rank; v += blockDim.x) o_lat[v] = merged_entry(w0, sstep, splits, comb_f, v);
+  __syncthreads();
+  const int end = min(vdim, ((int)blockIdx.y + 1) * LAT_UP_ROWS);
+  for (int j = blockIdx.y * LAT_UP_ROWS + warp; j < end; j += blockDim.x >> 5) {
+    const float v = row_dot(w_uv + ((size_t)h * vdim + j) * rank, o_lat, rank, lane, vec != 0);
+    if (lane == 0) st_act(out, (size_t)t * ldo + (size_t)h * vdim + j, v * (gate ? sigmoid_f(gate[(size_t)t * ldg + (size_t)h * vdim + j]) : 1.f));
+  }
+}
+
+// out[t, h * V + c] = in[t, h, c] * sigmoid(gate[t, h * V + c]): heads from any layout side by side, gated on the way.
+template <typename act_t>
+__global__ void seq_head_gate_kernel(const act_t* __restrict__ in, long long ld_t, long long ld_h, const float* __restrict__ gate, int ldg,
+                                     act_t* __restrict__ out, int ldo, int heads, int V) {
+  const int t = blockIdx.x;
+  for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < heads * V; i += gridDim.y * blockDim.x) {
+    const int h = i / V, c = i - h * V;
+    const float v = ld_act(in, (size_t)(t * ld_t + h * ld_h + c));
+    st_act(out, (size_t)t * ldo + i, gate ? v * sigmoid_f(gate[(size_t)t * ldg + i]) : v);
   }
 }
 
@@ -404,12 +555,13 @@ extern "C" int b2l_seq_latent_attention_warps(int T, int heads_per_group) {
 
 extern "C" int b2l_seq_latent_attention(const b2l_seq_latent_attn_args* a, b2l_stream_t stream) {
   B2L_CHECK_ARG(a != nullptr, "b2l_seq_latent_attention: null args");
-  B2L_CHECK_ARG(a->q_a && a->key_a && a->meta && a->out && (a->n_b == 0 || (a->q_b && a->key_b)), "b2l_seq_latent_attention: null pointer");
+  B2L_CHECK_ARG(a->q_a && a->key_a && a->meta && (a->out || a->partial) && (a->n_b == 0 || (a->q_b && a->key_b)), "b2l_seq_latent_attention: null pointer");
   B2L_CHECK_ARG(a->window >= 0, "b2l_seq_latent_attention: negative window");
   B2L_CHECK_ARG(a->T >= 0 && a->heads > 0 && a->heads_per_group > 0 && a->heads % a->heads_per_group == 0 && a->n_a > 0 && a->n_b >= 0 &&
                     a->vdim > 0 && a->vdim <= a->n_a && a->score_off >= 0 && a->score_off < a->n_a + a->n_b && a->score_off <= a->n_a &&
-                    a->splits >= 1 && a->ldo >= a->heads * a->vdim, "b2l_seq_latent_attention: bad size");
-  B2L_CHECK_ARG(a->splits == 1 || a->work, "b2l_seq_latent_attention: key splits need a workspace");
+                    a->splits >= 1 && (a->partial || a->ldo >= a->heads * a->vdim), "b2l_seq_latent_attention: bad size");
+  B2L_CHECK_ARG((a->splits == 1 && !a->partial) || a->work, "b2l_seq_latent_attention: key splits and partial results need a workspace");
+  B2L_CHECK_ARG(a->gate == nullptr || (!a->partial && a->ldg >= a->heads * a->vdim), "b2l_seq_latent_attention: bad gate");
   B2L_CHECK_SUPPORTED(a->splits <= 4096, "b2l_seq_latent_attention: %d key splits > 4096", a->splits);
   B2L_CHECK_SUPPORTED(a->vdim <= 512, "b2l_seq_latent_attention: value size %d > 512", a->vdim);
   if (a->T == 0) return 0;
@@ -428,12 +580,60 @@ extern "C" int b2l_seq_latent_attention(const b2l_seq_latent_attn_args* a, b2l_s
   });
   if (rc != 0) return rc;
   B2L_LAUNCH_CHECK("seq_latent_attention_kernel");
-  if (a->splits > 1) {
+  if (a->splits > 1 && !a->partial) {
     const int R = a->T * a->heads;
     B2L_SEQ_DISPATCH(a->act_dtype, {
-      seq_latent_combine_kernel<act_t><<<R, a->vdim > 128 ? 256 : 128, sizeof(float) * a->splits, st>>>(a->work, a->sink, (act_t*)a->out, a->ldo, R, a->heads, a->vdim, a->splits);
+      seq_latent_combine_kernel<act_t><<<R, a->vdim > 128 ? 256 : 128, sizeof(float) * a->splits, st>>>(a->work, a->sink, a->gate, a->ldg, (act_t*)a->out, a->ldo, R, a->heads,
+                                                                                                                a->vdim, a->splits);
     });
     B2L_LAUNCH_CHECK("seq_latent_combine_kernel");
   }
+  return 0;
+}
+
+extern "C" int b2l_seq_latent_operands(const b2l_seq_latent_operands_args* a, b2l_stream_t stream) {
+  B2L_CHECK_ARG(a != nullptr && a->proj && a->w_kv && a->meta && a->cache, "b2l_seq_latent_operands: null pointer");
+  B2L_CHECK_ARG(a->T >= 0 && a->heads > 0 && a->dn > 0 && a->dr >= 0 && a->rank > 0 && a->max_pos > 0 && a->q_off >= 0 && a->kv_off >= 0 &&
+                    a->ld >= a->q_off + a->heads * (a->dn + a->dr) && a->ld >= a->kv_off + a->rank + a->dr, "b2l_seq_latent_operands: bad size");
+  B2L_CHECK_ARG(a->rot_dims >= 0 && a->rot_dims <= a->dr && a->rot_dims % 2 == 0 && (a->rot_dims == 0 || a->freq), "b2l_seq_latent_operands: bad rotation");
+  B2L_CHECK_ARG((a->q_full != nullptr) + (a->q_nope != nullptr) + (a->q_lat != nullptr) == 1, "b2l_seq_latent_operands: one form of the queries is wanted");
+  B2L_CHECK_ARG(a->q_full || a->dr == 0 || a->q_rot, "b2l_seq_latent_operands: no place for the rotated queries");
+  B2L_CHECK_ARG(a->q_lat == nullptr || a->w_uk, "b2l_seq_latent_operands: latent queries need the key up-projection");
+  if (a->T == 0) return 0;
+  const int chunks = (a->rank + LAT_ABS_COLS - 1) / LAT_ABS_COLS;
+  const long long gy = 1 + (a->q_lat ? (long long)a->heads * chunks : 1);
+  const size_t smem = sizeof(float) * ((size_t)a->rot_dims + a->dn);
+  B2L_CHECK_SUPPORTED(gy <= 65535 && smem <= 40 * 1024, "b2l_seq_latent_operands: %d heads of %d + %d entries over a latent of %d are too many", a->heads, a->dn,
+                      a->dr, a->rank);
+  B2L_SEQ_DISPATCH(a->act_dtype, (seq_latent_operands_kernel<act_t><<<dim3(a->T, (unsigned)gy), 256, smem, (cudaStream_t)stream>>>(*a, chunks)));
+  B2L_LAUNCH_CHECK("seq_latent_operands_kernel");
+  return 0;
+}
+
+extern "C" int b2l_seq_latent_up(const float* work, const float* sink, const void* w_uv, const float* gate, int ldg, void* out, int ldo, int T, int heads,
+                                 int rank, int vdim, int splits, int act_dtype, b2l_stream_t stream) {
+  B2L_CHECK_ARG(work && w_uv && out, "b2l_seq_latent_up: null pointer");
+  B2L_CHECK_ARG(T >= 0 && heads > 0 && rank > 0 && vdim > 0 && splits >= 1 && ldo >= heads * vdim && (!gate || ldg >= heads * vdim), "b2l_seq_latent_up: bad size");
+  const size_t smem = sizeof(float) * ((size_t)rank + splits);
+  B2L_CHECK_SUPPORTED(smem <= 48 * 1024, "b2l_seq_latent_up: a latent of %d entries and %d key splits need %zu bytes of shared memory", rank, splits, smem);
+  if (T == 0) return 0;
+  B2L_SEQ_DISPATCH(act_dtype, {
+    constexpr int PER = 16 / sizeof(act_t);
+    seq_latent_up_kernel<act_t><<<dim3(T * heads, (vdim + LAT_UP_ROWS - 1) / LAT_UP_ROWS), 256, smem, (cudaStream_t)stream>>>(
+        work, sink, (const act_t*)w_uv, gate, ldg, (act_t*)out, ldo, T * heads, heads, rank, vdim, splits, rank % PER == 0 && al16(w_uv));
+  });
+  B2L_LAUNCH_CHECK("seq_latent_up_kernel");
+  return 0;
+}
+
+extern "C" int b2l_seq_head_gate(const void* in, long long ld_t, long long ld_h, const float* gate, int ldg, void* out, int ldo, int T, int heads, int V,
+                                 int act_dtype, b2l_stream_t stream) {
+  B2L_CHECK_ARG(in && out && in != out, "b2l_seq_head_gate: null pointer, or the output is the input");
+  B2L_CHECK_ARG(T >= 0 && heads > 0 && V > 0 && ldo >= heads * V && (!gate || ldg >= heads * V), "b2l_seq_head_gate: bad size");
+  if (T == 0) return 0;
+  const int gy = (heads * V + 255) / 256;
+  B2L_SEQ_DISPATCH(act_dtype, (seq_head_gate_kernel<act_t><<<dim3(T, gy < 64 ? gy : 64), 256, 0, (cudaStream_t)stream>>>((const act_t*)in, ld_t, ld_h, gate, ldg,
+                                                                                                                       (act_t*)out, ldo, heads, V)));
+  B2L_LAUNCH_CHECK("seq_head_gate_kernel");
   return 0;
 }

@@ -1,6 +1,6 @@
 // Mixture-of-experts feed-forward: the router (softmax or sigmoid scores, a selection bias that only steers the choice,
 // groups of neighbouring experts of which only the best may be chosen, top-k, weights renormalised over the chosen or
-// the scores themselves; the weight scales an expert's output or its input), the
+// the scores themselves, or a softmax over the chosen logits alone; the weight scales an expert's output or its input), the
 // expert products for a handful of tokens with the expert index read on the device (a captured single-token step
 // replays for any routing), and the sort / gather / combine around the per-expert library products of long portions.
 // Experts with index >= n_real are identities: their output is the input itself.
@@ -36,6 +36,14 @@ __device__ __forceinline__ void route_token(const float* zr, const float* __rest
       s[i] = sigmoid_f(zr[i]);
       c[i] = s[i] + (corr ? corr[i] : 0.f);
     }
+  } else if (score_fn == B2L_SEQ_SCORE_CHOSEN_SOFTMAX) {        // the choice is made on the logits themselves
+    float mx = -INFINITY;
+    for (int i = lane; i < n; i += 32) {
+      c[i] = zr[i] + (corr ? corr[i] : 0.f);
+      mx = fmaxf(mx, c[i]);
+    }
+    mx = warp_max(mx);
+    for (int i = lane; i < n; i += 32) s[i] = expf(c[i] - mx);
   } else {
     float mx = -INFINITY;
     for (int i = lane; i < n; i += 32) mx = fmaxf(mx, zr[i]);
@@ -120,34 +128,6 @@ __global__ void seq_moe_route_kernel(const float* __restrict__ z, int ldz, const
               lane);
 }
 
-// Dot product of a weight row with a vector in shared memory (f32); the warp's lanes stride the row.
-template <typename act_t>
-__device__ __forceinline__ float row_dot(const act_t* __restrict__ w, const float* __restrict__ x, int n, int lane, bool vec) {
-  float acc = 0.f;
-  if (vec) {                                         // 16-byte loads: n a multiple of 8 (bf16) / 4 (f32), aligned rows
-    constexpr int PER = 16 / sizeof(act_t);
-    for (int i = lane * PER; i < n; i += 32 * PER) {
-      const uint4 u = *reinterpret_cast<const uint4*>(w + i);
-      if (sizeof(act_t) == 2) {
-        const uint32_t ww[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-        for (int q = 0; q < 4; ++q) {
-          acc = fmaf(__uint_as_float(ww[q] << 16), x[i + 2 * q], acc);
-          acc = fmaf(__uint_as_float(ww[q] & 0xffff0000u), x[i + 2 * q + 1], acc);
-        }
-      } else {
-        acc = fmaf(__uint_as_float(u.x), x[i], acc);
-        acc = fmaf(__uint_as_float(u.y), x[i + 1], acc);
-        acc = fmaf(__uint_as_float(u.z), x[i + 2], acc);
-        acc = fmaf(__uint_as_float(u.w), x[i + 3], acc);
-      }
-    }
-  } else {
-    for (int i = lane; i < n; i += 32) acc = fmaf(ld_act(w, i), x[i], acc);
-  }
-  return warp_sum(acc);
-}
-
 // Router of a few tokens in one launch: the logits W_router h_t (f32 accumulation of exact products; a warp per
 // router row) and the routing.  One CTA per token.  Shared: x[D], z[n], s[n], c[n], g[groups].
 template <typename act_t>
@@ -170,18 +150,34 @@ __global__ void __launch_bounds__(1024) seq_moe_route_fused_kernel(const act_t* 
     route_token(z, corr, n, groups, keep, top, score_fn, renorm, group_top, weight_scale, idx + (size_t)t * top, wgt + (size_t)t * top, z + n, z + 2 * n, z + 3 * n, lane);
 }
 
+// An expert that every token uses beside its chosen ones (ff == 0: none): W_down (gated(W_gate h, W_up h)), unweighted.
+template <typename act_t>
+struct SharedExpert {
+  const act_t* gu;      // [2*ff][D]
+  const act_t* down;    // [D][ff]
+  act_t* mid;           // [T][ff]
+  int ff, vec_dn;
+};
+
 // mid[a, j] = gated(W_gate[e] x, W_up[e] x) for assignment a = t * top + k, e = idx[a], x = h_t or (in_scale given) the
-// storage-type rounding of in_scale[a] * h_t.  grid (N, ff chunks).
+// storage-type rounding of in_scale[a] * h_t.  grid (N (+ T with a shared expert), ff chunks).
 template <typename act_t>
 __global__ void __launch_bounds__(256) seq_moe_up_kernel(const act_t* __restrict__ h, int ldh, const act_t* __restrict__ wgu,
                                                          const int* __restrict__ idx, const float* __restrict__ in_scale,
                                                          act_t* __restrict__ mid, int D, int ff, int n_real, int top, int act, float limit,
-                                                         int vec) {
+                                                         int vec, int N, SharedExpert<act_t> sh) {
   extern __shared__ float moe_x[];
-  const int a = blockIdx.x, e = idx[a];
-  if (e >= n_real) return;
-  const act_t* hr = h + (size_t)(a / top) * ldh;
-  if (in_scale) {
+  const int a = blockIdx.x, wpc = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const bool shared = a >= N;
+  const int e = shared ? 0 : idx[a], t = shared ? a - N : a / top;
+  if (!shared) {
+    if (e >= n_real) return;
+  } else {
+    ff = sh.ff;
+  }
+  if ((int)blockIdx.y * wpc >= ff) return;           // the grid covers the wider of the two kinds
+  const act_t* hr = h + (size_t)t * ldh;
+  if (in_scale && !shared) {
     const float w = in_scale[a];
     for (int i = threadIdx.x; i < D; i += blockDim.x) {
       act_t tmp[1];
@@ -192,8 +188,8 @@ __global__ void __launch_bounds__(256) seq_moe_up_kernel(const act_t* __restrict
     for (int i = threadIdx.x; i < D; i += blockDim.x) moe_x[i] = ld_act(hr, i);
   }
   __syncthreads();
-  const int wpc = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const act_t* w = wgu + (size_t)e * 2 * ff * D;
+  const act_t* w = shared ? sh.gu : wgu + (size_t)e * 2 * ff * D;
+  act_t* m = shared ? sh.mid + (size_t)t * ff : mid + (size_t)a * ff;
   for (int j = blockIdx.y * wpc + warp; j < ff; j += gridDim.y * wpc) {
     const float gv = row_dot(w + (size_t)j * D, moe_x, D, lane, vec);
     const float uv = row_dot(w + (size_t)(ff + j) * D, moe_x, D, lane, vec);
@@ -202,23 +198,27 @@ __global__ void __launch_bounds__(256) seq_moe_up_kernel(const act_t* __restrict
       act_t tmp[2];
       st_act(tmp, 0, gv);
       st_act(tmp, 1, uv);
-      st_act(mid, (size_t)a * ff + j, gated_pair(ld_act(tmp, 0), ld_act(tmp, 1), act, limit));
+      st_act(m, j, gated_pair(ld_act(tmp, 0), ld_act(tmp, 1), act, limit));
     }
   }
 }
 
-// y[t, i] = sum_k w[t, k] * (e < n_real ? W_down[e][i, :] . mid[a, :] : h[t, i]).  grid (T, D chunks).
+// y[t, i] = sum_k w[t, k] * (e < n_real ? W_down[e][i, :] . mid[a, :] : h[t, i]), plus the shared expert's output.
+// grid (T, D chunks).
 template <typename act_t>
 __global__ void __launch_bounds__(256) seq_moe_down_kernel(const act_t* __restrict__ mid, const act_t* __restrict__ wd,
                                                            const int* __restrict__ idx, const float* __restrict__ wgt,
                                                            const float* __restrict__ in_scale, const act_t* __restrict__ h, int ldh,
-                                                           act_t* __restrict__ y, int ldy, int D, int ff, int n_real, int top, int vec) {
+                                                           act_t* __restrict__ y, int ldy, int D, int ff, int n_real, int top, int vec,
+                                                           SharedExpert<act_t> sh) {
   extern __shared__ float moe_x[];
   const int t = blockIdx.x;
   for (int i = threadIdx.x; i < top * ff; i += blockDim.x) {
     const int k = i / ff;
     moe_x[i] = idx[(size_t)t * top + k] < n_real ? ld_act(mid, ((size_t)t * top + k) * ff + (i % ff)) : 0.f;
   }
+  float* moe_s = moe_x + ((top * ff + 3) & ~3);
+  for (int i = threadIdx.x; i < sh.ff; i += blockDim.x) moe_s[i] = ld_act(sh.mid, (size_t)t * sh.ff + i);
   __syncthreads();
   const int wpc = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   for (int i = blockIdx.y * wpc + warp; i < D; i += gridDim.y * wpc) {
@@ -236,6 +236,11 @@ __global__ void __launch_bounds__(256) seq_moe_down_kernel(const act_t* __restri
         v = ld_act(h, (size_t)t * ldh + i) * ((wgt || in_scale == nullptr) ? 1.f : in_scale[(size_t)t * top + k]);
       }
       acc = fmaf(wk, v, acc);
+    }
+    if (sh.ff > 0) {
+      act_t tmp[1];
+      st_act(tmp, 0, row_dot(sh.down + (size_t)i * sh.ff, moe_s, sh.ff, lane, sh.vec_dn != 0));
+      acc += ld_act(tmp, 0);
     }
     if (lane == 0) st_act(y, (size_t)t * ldy + i, acc);
   }
@@ -286,13 +291,14 @@ __global__ void seq_moe_gather_kernel(const act_t* __restrict__ h, int ldh, cons
     for (int i = threadIdx.x; i < D; i += blockDim.x) dst[i] = src[i];
   }
 }
-// y[t, i] = sum_k w[t, k] * (inv[a] >= 0 ? yg[inv[a], i] : h[t, i]).  One CTA per token.
+// y[t, i] = sum_k w[t, k] * (inv[a] >= 0 ? yg[inv[a], i] : h[t, i]) (+ add[t, i]).  One CTA per token.
 template <typename act_t>
 __global__ void seq_moe_combine_kernel(const act_t* __restrict__ yg, const int* __restrict__ inv, const float* __restrict__ wgt,
-                                       const act_t* __restrict__ h, int ldh, act_t* __restrict__ y, int ldy, int D, int top) {
+                                       const act_t* __restrict__ h, int ldh, const act_t* __restrict__ add, int ldadd, act_t* __restrict__ y,
+                                       int ldy, int D, int top) {
   const int t = blockIdx.x;
   for (int i = threadIdx.x; i < D; i += blockDim.x) {
-    float acc = 0.f;
+    float acc = add ? ld_act(add, (size_t)t * ldadd + i) : 0.f;
     for (int k = 0; k < top; ++k) {
       const int p = inv[(size_t)t * top + k];
       const float v = p >= 0 ? ld_act(yg, (size_t)p * D + i) : ld_act(h, (size_t)t * ldh + i);
@@ -315,7 +321,8 @@ extern "C" int b2l_seq_moe_route(const float* logits, int ld, const float* corre
   B2L_CHECK_ARG(T >= 0 && n > 0 && ld >= n && top > 0 && top <= n && groups >= 1 && n % groups == 0 && keep >= 1 && keep <= groups,
                 "b2l_seq_moe_route: bad size");
   B2L_CHECK_ARG((long long)keep * (n / groups) >= top, "b2l_seq_moe_route: the kept groups hold fewer than `top` experts");
-  B2L_CHECK_ARG(score_fn == B2L_SEQ_SCORE_SOFTMAX || score_fn == B2L_SEQ_SCORE_SIGMOID, "b2l_seq_moe_route: unknown score function %d", score_fn);
+  B2L_CHECK_ARG(score_fn >= B2L_SEQ_SCORE_SOFTMAX && score_fn <= B2L_SEQ_SCORE_CHOSEN_SOFTMAX, "b2l_seq_moe_route: unknown score function %d", score_fn);
+  B2L_CHECK_ARG(score_fn != B2L_SEQ_SCORE_CHOSEN_SOFTMAX || renormalize, "b2l_seq_moe_route: a softmax over the chosen logits is renormalised by definition");
   if (T == 0) return 0;
   const int wpc = 4;
   const size_t smem = sizeof(float) * wpc * (2 * (size_t)n + groups);
@@ -326,8 +333,6 @@ extern "C" int b2l_seq_moe_route(const float* logits, int ld, const float* corre
   return 0;
 }
 
-static inline bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; }
-
 extern "C" int b2l_seq_moe_route_fused(const void* h, int ldh, const void* w_router, const float* correction, int D, int n, int groups,
                                        int keep, int top, int score_fn, int renormalize, int group_top, float weight_scale, int* idx,
                                        float* weights, int T, int act_dtype, b2l_stream_t stream) {
@@ -336,7 +341,8 @@ extern "C" int b2l_seq_moe_route_fused(const void* h, int ldh, const void* w_rou
   B2L_CHECK_ARG(T >= 0 && D > 0 && ldh >= D && n > 0 && top > 0 && top <= n && groups >= 1 && n % groups == 0 && keep >= 1 && keep <= groups,
                 "b2l_seq_moe_route_fused: bad size");
   B2L_CHECK_ARG((long long)keep * (n / groups) >= top, "b2l_seq_moe_route_fused: the kept groups hold fewer than `top` experts");
-  B2L_CHECK_ARG(score_fn == B2L_SEQ_SCORE_SOFTMAX || score_fn == B2L_SEQ_SCORE_SIGMOID, "b2l_seq_moe_route_fused: unknown score function %d", score_fn);
+  B2L_CHECK_ARG(score_fn >= B2L_SEQ_SCORE_SOFTMAX && score_fn <= B2L_SEQ_SCORE_CHOSEN_SOFTMAX, "b2l_seq_moe_route_fused: unknown score function %d", score_fn);
+  B2L_CHECK_ARG(score_fn != B2L_SEQ_SCORE_CHOSEN_SOFTMAX || renormalize, "b2l_seq_moe_route_fused: a softmax over the chosen logits is renormalised by definition");
   if (T == 0) return 0;
   const size_t smem = sizeof(float) * ((size_t)D + 3 * (size_t)n + groups);
   B2L_CHECK_SUPPORTED(smem <= 200 * 1024, "b2l_seq_moe_route_fused: width %d and %d experts need %zu bytes of shared memory", D, n, smem);
@@ -355,14 +361,16 @@ extern "C" int b2l_seq_moe_route_fused(const void* h, int ldh, const void* w_rou
 
 extern "C" int b2l_seq_moe_experts_small(const void* h, int ldh, const void* w_gate_up, const void* w_down, const int* idx,
                                          const float* weights, void* mid, void* y, int ldy, int T, int D, int ff, int n_real,
-                                         int top, int act, float limit, int weight_input, int act_dtype, b2l_stream_t stream) {
+                                         int top, int act, float limit, int weight_input, const void* w_shared_gate_up, const void* w_shared_down,
+                                         int ff_shared, int act_dtype, b2l_stream_t stream) {
   B2L_CHECK_ARG(h && idx && weights && mid && y && (n_real == 0 || (w_gate_up && w_down)), "b2l_seq_moe_experts_small: null pointer");
+  B2L_CHECK_ARG(ff_shared >= 0 && (ff_shared == 0 || (w_shared_gate_up && w_shared_down)), "b2l_seq_moe_experts_small: bad shared expert");
   B2L_CHECK_ARG(T >= 0 && D > 0 && ff > 0 && top > 0 && n_real >= 0 && ldh >= D && ldy >= D, "b2l_seq_moe_experts_small: bad size");
   B2L_CHECK_ARG(act >= 0 && act <= 3 && (act != B2L_SEQ_ACT_CLAMPED_SWISH || limit > 0.f), "b2l_seq_moe_experts_small: bad activation");
   if (T == 0) return 0;
   cudaStream_t st = (cudaStream_t)stream;
-  const size_t smem_up = sizeof(float) * (size_t)D, smem_dn = sizeof(float) * (size_t)top * ff;
-  B2L_CHECK_SUPPORTED(smem_up <= 200 * 1024 && smem_dn <= 200 * 1024, "b2l_seq_moe_experts_small: width %d or top * ff %d too large", D, top * ff);
+  const size_t smem_up = sizeof(float) * (size_t)D, smem_dn = sizeof(float) * ((((size_t)top * ff + 3) & ~(size_t)3) + ff_shared);
+  B2L_CHECK_SUPPORTED(smem_up <= 200 * 1024 && smem_dn <= 200 * 1024, "b2l_seq_moe_experts_small: width %d, top * ff %d or shared ff %d too large", D, top * ff, ff_shared);
   B2L_SEQ_DISPATCH(act_dtype, {
     constexpr int PER = 16 / sizeof(act_t);
     const int vec_up = (D % PER == 0 && al16(w_gate_up)) ? 1 : 0;
@@ -371,13 +379,16 @@ extern "C" int b2l_seq_moe_experts_small(const void* h, int ldh, const void* w_g
     if (rc != 0) return rc;
     rc = ensure_dyn_smem(seq_moe_down_kernel<act_t>, smem_dn, g_moe_smem[sizeof(act_t) == 2 ? 2 : 3]);
     if (rc != 0) return rc;
-    if (n_real > 0)
-      seq_moe_up_kernel<act_t><<<dim3(T * top, (ff + 7) / 8), 256, smem_up, st>>>((const act_t*)h, ldh, (const act_t*)w_gate_up, idx,
-                                                                                   weight_input ? weights : nullptr, (act_t*)mid, D, ff, n_real,
-                                                                                   top, act, limit, vec_up);
+    const int N = T * top, ff_max = ff_shared > ff ? ff_shared : ff;
+    SharedExpert<act_t> sh{(const act_t*)w_shared_gate_up, (const act_t*)w_shared_down, (act_t*)mid + (size_t)N * ff, ff_shared,
+                           (ff_shared % PER == 0 && al16(w_shared_down)) ? 1 : 0};
+    if (n_real > 0 || ff_shared > 0)
+      seq_moe_up_kernel<act_t><<<dim3(N + (ff_shared > 0 ? T : 0), (ff_max + 7) / 8), 256, smem_up, st>>>(
+          (const act_t*)h, ldh, (const act_t*)w_gate_up, idx, weight_input ? weights : nullptr, (act_t*)mid, D, ff, n_real, top, act, limit,
+          vec_up && (ff_shared == 0 || al16(w_shared_gate_up)), N, sh);
     seq_moe_down_kernel<act_t><<<dim3(T, (D + 7) / 8), 256, smem_dn, st>>>((const act_t*)mid, (const act_t*)w_down, idx,
                                                                             weight_input ? nullptr : weights, weight_input ? weights : nullptr,
-                                                                            (const act_t*)h, ldh, (act_t*)y, ldy, D, ff, n_real, top, vec_dn);
+                                                                            (const act_t*)h, ldh, (act_t*)y, ldy, D, ff, n_real, top, vec_dn, sh);
   });
   B2L_LAUNCH_CHECK("seq_moe_up_kernel / seq_moe_down_kernel");
   return 0;
@@ -408,13 +419,14 @@ extern "C" int b2l_seq_moe_gather(const void* h, int ldh, const int* perm, const
   return 0;
 }
 
-extern "C" int b2l_seq_moe_combine(const void* yg, const int* inv, const float* weights, const void* h, int ldh, void* y, int ldy,
-                                   int T, int D, int top, int act_dtype, b2l_stream_t stream) {
+extern "C" int b2l_seq_moe_combine(const void* yg, const int* inv, const float* weights, const void* h, int ldh, const void* add,
+                                   int ldadd, void* y, int ldy, int T, int D, int top, int act_dtype, b2l_stream_t stream) {
   B2L_CHECK_ARG(yg && inv && h && y, "b2l_seq_moe_combine: null pointer");
-  B2L_CHECK_ARG(T >= 0 && D > 0 && top > 0 && ldh >= D && ldy >= D, "b2l_seq_moe_combine: bad size");
+  B2L_CHECK_ARG(T >= 0 && D > 0 && top > 0 && ldh >= D && ldy >= D && (!add || ldadd >= D), "b2l_seq_moe_combine: bad size");
   if (T == 0) return 0;
   B2L_SEQ_DISPATCH(act_dtype, {
-    seq_moe_combine_kernel<act_t><<<T, 256, 0, (cudaStream_t)stream>>>((const act_t*)yg, inv, weights, (const act_t*)h, ldh, (act_t*)y, ldy, D, top);
+    seq_moe_combine_kernel<act_t><<<T, 256, 0, (cudaStream_t)stream>>>((const act_t*)yg, inv, weights, (const act_t*)h, ldh, (const act_t*)add, ldadd, (act_t*)y, ldy,
+                                                                    D, top);
   });
   B2L_LAUNCH_CHECK("seq_moe_combine_kernel");
   return 0;

@@ -140,6 +140,7 @@ __global__ void seq_scale_kernel(float* __restrict__ z, size_t n, float mult) {
 //   entries of every head (entry i with entry i + rot_dims/2) by the angle (pos0 + t) * freq[i]; unit_rms (no weights): the
 //   rotated head divided by its root mean square.  A rotation keeps the length of the pairs it turns up to rot_mult, so
 //   the sum of squares is taken from the entries before it.
+//   q_out is multiplied by the query temperature of its position when temp_every > 0.
 //   v_out (act): (1 - lambda) v + lambda v_first when v_first is given (lambda read on the device), else not written.
 template <typename act_t>
 __global__ void __launch_bounds__(256) seq_qkv_prep_kernel(b2l_seq_qkv_prep_args a) {
@@ -148,6 +149,7 @@ __global__ void __launch_bounds__(256) seq_qkv_prep_kernel(b2l_seq_qkv_prep_args
   const act_t* row = (const act_t*)a.proj + (size_t)t * a.ld;
   const float pos = (float)(a.meta[1] + t);
   const int half = a.rot_dims / 2, K = a.K;
+  const float temp = a.temp_every > 0 ? 1.0f + a.temp_coef * logf((float)((a.meta[1] + t + 1) / a.temp_every + 1)) : 1.0f;
   for (int which = 0; which < 2; ++which) {
     const act_t* x = row + (which == 0 ? a.q_off : a.k_off);
     const act_t* w = (const act_t*)(which == 0 ? a.q_norm : a.k_norm);
@@ -186,8 +188,8 @@ __global__ void __launch_bounds__(256) seq_qkv_prep_kernel(b2l_seq_qkv_prep_args
         s *= a.rot_mult;
         c *= a.rot_mult;
         if (which == 0) {
-          qo[i] = u * c - v * s;
-          qo[i + half] = v * c + u * s;
+          qo[i] = (u * c - v * s) * temp;
+          qo[i + half] = (v * c + u * s) * temp;
         } else {
           st_act(ko, i, u * c - v * s);
           st_act(ko, i + half, v * c + u * s);
@@ -195,7 +197,7 @@ __global__ void __launch_bounds__(256) seq_qkv_prep_kernel(b2l_seq_qkv_prep_args
       }
       for (int i = a.rot_dims + lane; i < K; i += 32) {
         const float v = ld_act(p, i) * r * (wh ? ld_act(wh, i) : 1.f);
-        if (which == 0) qo[i] = v;
+        if (which == 0) qo[i] = v * temp;
         else st_act(ko, i, v);
       }
     }
@@ -297,6 +299,7 @@ extern "C" int b2l_seq_qkv_prep(const b2l_seq_qkv_prep_args* a, b2l_stream_t str
   B2L_CHECK_ARG(a->T >= 0 && a->heads > 0 && a->kv_heads > 0 && a->K > 0 && a->V > 0, "b2l_seq_qkv_prep: bad size");
   B2L_CHECK_ARG(a->rot_dims >= 0 && a->rot_dims <= a->K && a->rot_dims % 2 == 0 && (a->rot_dims == 0 || a->freq), "b2l_seq_qkv_prep: bad rotation");
   B2L_CHECK_ARG((a->v_first == nullptr) || (a->v_out && a->lambda), "b2l_seq_qkv_prep: value mixing needs lambda and an output");
+  B2L_CHECK_ARG(a->temp_every >= 0, "b2l_seq_qkv_prep: negative temperature step");
   B2L_CHECK_ARG(!a->unit_rms || (a->q_norm == nullptr && a->k_norm == nullptr), "b2l_seq_qkv_prep: the norm after the rotation has no weight");
   if (a->T == 0) return 0;
   B2L_SEQ_DISPATCH(a->act_dtype, (seq_qkv_prep_kernel<act_t><<<a->T, 256, 0, (cudaStream_t)stream>>>(*a)));

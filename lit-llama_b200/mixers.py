@@ -9,14 +9,17 @@ constants are constructor parameters.
     ParallelMixer        two mixers on the same input, one output product over their concatenated read-outs
     Mamba2Mixer          state-space duality layer: scalar decay per head, convolution on x | B | C, gated grouped norm
     LatentAttention      causal softmax attention whose keys and values are linear images of one cached latent per position
-                         (+ one rotated key part shared by the heads), low-rank queries, a learned sink per head
+                         (+ one rotated key part shared by the heads), low-rank or direct queries, a learned sink per head,
+                         an optional sigmoid gate per output channel
     RetentionMixer       linear attention with a fixed decay per head, rotated q / k, per-head unit-RMS read-out, silu gate
-    MoEFeedForward       routed gated experts: softmax or sigmoid scores, selection bias, expert groups, top-k, identity
-                         experts, weights renormalised or not, on an expert's output or on its input, clamped gated unit
+    MoEFeedForward       routed gated experts: softmax or sigmoid scores or a softmax over the chosen logits, selection or logit
+                         bias, expert groups, top-k, identity experts, a shared expert, weights renormalised or not, on an
+                         expert's output or on its input, clamped gated unit
     LocalAttention       causal softmax attention over the last `window` positions (SlidingWindowAttention) or inside blocks:
                          q/k norm over the whole projection or per head before the rotation, or weightless per head after it,
-                         partial rotation, grouped kv heads, values mixed with an earlier layer's, an optional sigmoid gate per
-                         output channel, ring cache of one window or block
+                         partial rotation, a query temperature by position, grouped kv heads, values mixed with an earlier
+                         layer's, an optional one in the softmax denominator, an optional sigmoid gate per head or per output
+                         channel, ring cache of one window or block
     PairHashEmbedding    token embedding plus a hashed (previous token, token) embedding, into several residual streams
     HyperConnection      one sublayer's read weights, stream-mixing matrix and write weights over several residual streams
     DenseMLP             W_down act(W_up h) without a gate: gelu_tanh, silu, relu2, or xIELU with its two learned numbers
@@ -25,6 +28,8 @@ constants are constructor parameters.
                          interleaved rotation, grouped kv heads, keys and values of its own or of an earlier layer
     MinGRUMixer          S_t = (1 - z_t) S_(t-1) + z_t c_t per channel with gates that read only the current token, silu gate
     DepthAverage         the residual step of layers whose input is a learned average over all earlier layers' results
+    residual_step        x + results (+ a vector, + an f32 row), fused with the next norm or with the operand of a product on x
+    LoopInjection        what a looped stretch of layers reads: x <- W [x; embedding output] + a vector of the pass
     MatrixMemoryMixer    mLSTM: a matrix state per head with exponential input gates, sigmoid forget gates, a normaliser and a
                          running maximum; per-head unit-RMS read-out, one weight, a sigmoid gate per channel
     share_weights        the same mixer over the same weights with a state of its own (a layer that runs again)
@@ -96,6 +101,9 @@ def share_weights(mixer, name: str):
     twin = copy.copy(mixer)
     twin.name = name
     return twin
+
+
+FEW_TOKENS = 4          # up to this many tokens a mechanism may run its products in its own kernels, without the library
 
 
 def linear(x: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
@@ -529,9 +537,11 @@ class LocalAttention:
         rotation of the first rot.dims entries of every head (entry i with entry i + dims/2); or ("unit") the rotation first,
         then every head divided by its root mean square, without a weight
         v <- (1 - lambda) v + lambda v_first in every layer with `v_mix` but the first of them, whose v is v_first
-        weights = softmax(q . k * scale) over the visible keys (ordinary softmax, no sink); query head h reads
-        key / value head h // (heads / kv_heads)
-        y = W_o (concat_h(sum_j weight_j v_j) * sigmoid(W_g h))            a gate per output channel; no gate when not `gate`
+        with `q_temp` = {"coef", "every"} q at position p is multiplied by 1 + coef ln(floor((p + 1) / every) + 1)
+        weights = softmax(q . k * scale) over the visible keys, with `sink` exp(s_j) / (1 + sum_j exp(s_j)); query head h
+        reads key / value head h // (heads / kv_heads)
+        y = W_o (concat_h(sum_j weight_j v_j) * sigmoid(W_g h))            a gate per output channel (`gate` = "channel" or
+        True), one number per head (`gate` = "head"), or no gate (False)
 
     State per sequence: a ring of `window` (or `block`) positions of rotated keys and (mixed) values, entry position %
     size.  The first value-mixing layer of a step leaves its values in `ctx.shared` for the later ones."""
@@ -540,7 +550,8 @@ class LocalAttention:
 
     def __init__(self, name: str, W: Dict[str, torch.Tensor], p: str, *, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float,
                  window: Optional[int] = None, block: Optional[int] = None, max_positions: int = 0, rot: Optional[dict] = None,
-                 norm_over: str = "row", gate: bool = True, v_mix: bool = False, mix_key: str = "v_first") -> None:
+                 norm_over: str = "row", gate=True, v_mix: bool = False, mix_key: str = "v_first", sink: bool = False,
+                 q_temp: Optional[dict] = None) -> None:
         self.name, self.H, self.G, self.K, self.V, self.scale, self.eps = name, int(heads), int(kv_heads), int(dim), int(vdim), float(scale), eps
         if window is not None and block is not None:
             raise ValueError("local attention: a window or blocks, not both")
@@ -553,7 +564,14 @@ class LocalAttention:
         self.whole_row, self.unit_rms, self.v_mix, self.mix_key = int(norm_over == "row"), int(norm_over == "unit"), bool(v_mix), mix_key
         assert W[p + "q"].shape[0] == heads * dim and W[p + "k"].shape[0] == kv_heads * dim and W[p + "v"].shape[0] == kv_heads * vdim, \
             "local attention: projections do not fit the head sizes"
-        assert W[p + "o"].shape[1] == heads * vdim and (not gate or W[p + "g"].shape[0] == heads * vdim), "local attention: gate / output do not fit"
+        if gate not in (True, False, "channel", "head"):
+            raise ValueError(f"local attention: gate per {gate!r}")
+        self.gate_per_channel, self.sink = int(gate in (True, "channel")), int(bool(sink))
+        assert W[p + "o"].shape[1] == heads * vdim and (not gate or W[p + "g"].shape[0] == (heads * vdim if self.gate_per_channel else heads)), \
+            "local attention: gate / output do not fit"
+        self.temp_coef, self.temp_every = (float(q_temp["coef"]), int(q_temp["every"])) if q_temp else (0.0, 0)
+        if q_temp and (self.temp_every < 1 or self.temp_every != q_temp["every"]):
+            raise ValueError(f"local attention: the query temperature steps every {q_temp['every']!r} positions")
         self.w_in, offs = stack_rows([W[p + "q"], W[p + "k"], W[p + "v"]] + ([W[p + "g"]] if gate else []))
         self.o_q, self.o_k, self.o_v = offs[:3]
         self.o_g = offs[3] if gate else None
@@ -592,14 +610,15 @@ class LocalAttention:
                           whole_row=self.whole_row, eps=self.eps, freq=_p(self.freq), rot_dims=self.rot_dims, rot_mult=self.rot_mult,
                           meta=_p(ctx.meta), q_out=_p(q), k_out=_p(kn), v_first=_p(first[0], first[1]) if first is not None else None,
                           ldvf=first[2] if first is not None else 0, lambda_=_p(self.lam) if first is not None else None, v_out=_p(vm), T=T,
-                          heads=self.H, kv_heads=self.G, K=self.K, V=self.V, act_dtype=ctx.act, unit_rms=self.unit_rms)
+                          heads=self.H, kv_heads=self.G, K=self.K, V=self.V, act_dtype=ctx.act, unit_rms=self.unit_rms, temp_coef=self.temp_coef,
+                          temp_every=self.temp_every)
         S.check(lib.b2l_seq_qkv_prep(C.byref(a), ctx.stream), "b2l_seq_qkv_prep")
         att = torch.empty((T, self.H * self.V), dtype=h.dtype, device=dev)
         gated = self.o_g is not None
         b = S.AttnArgs(q=_p(q), k_new=_p(kn), v_new=_p(v, v_off), ldv=ldv, cache_k=_p(ctx.state[self.name + ".k"]),
                        cache_v=_p(ctx.state[self.name + ".v"]), meta=_p(ctx.meta), gate=_p(proj, self.o_g) if gated else None, ldg=ld if gated else 0,
-                       out=_p(att), ldo=self.H * self.V, scale=self.scale, softcap=0.0, out_mult=1.0, has_sink=0, block=self.ring, T=T, heads=self.H,
-                       kv_heads=self.G, K=self.K, V=self.V, act_dtype=ctx.act, window=self.window, gate_per_channel=int(gated))
+                       out=_p(att), ldo=self.H * self.V, scale=self.scale, softcap=0.0, out_mult=1.0, has_sink=self.sink, block=self.ring, T=T, heads=self.H,
+                       kv_heads=self.G, K=self.K, V=self.V, act_dtype=ctx.act, window=self.window, gate_per_channel=self.gate_per_channel)
         local_attention(b, ctx)
         return linear(att, self.w_o)
 
@@ -712,8 +731,69 @@ def norm_rows(x: torch.Tensor, w: torch.Tensor, b: Optional[torch.Tensor], kind:
     """RMS norm ("rms") or layer norm with a bias ("layer") of rows of the f32 stream x [T, width] -> act [n_rows, width]."""
     n = x.shape[0] if n_rows is None else n_rows
     out = torch.empty((n, x.shape[1]), dtype=ctx.dtype, device=x.device)
-    S.check(S.lib().b2l_seq_norm(_p(x), _p(w), _p(b), DepthAverage.NORMS[kind], eps, _p(out), _p(rows), n, x.shape[1], ctx.act, ctx.stream), "b2l_seq_norm")
+    S.check(S.lib().b2l_seq_norm(_p(x), _p(w), _p(b), NORM_KINDS[kind], eps, _p(out), _p(rows), n, x.shape[1], ctx.act, ctx.stream), "b2l_seq_norm")
     return out
+
+
+NORM_KINDS = {"rms": S.NORM_RMS, "layer": S.NORM_LAYER}
+
+
+def residual_step(x_in: torch.Tensor, x_out: Optional[torch.Tensor], ctx: StepContext, *, y1: Optional[torch.Tensor] = None, y2: Optional[torch.Tensor] = None,
+                  vec: Optional[torch.Tensor] = None, base: Optional[torch.Tensor] = None, norm: Optional[torch.Tensor] = None,
+                  bias: Optional[torch.Tensor] = None, kind: str = "rms", eps: float = 0.0, split: bool = False) -> Optional[torch.Tensor]:
+    """x_out = x_in + y1 + y2 (act rows) + vec (act, the same for every token) + base (f32 rows), f32 [T, width]; x_out may be
+    x_in.  Returns norm(x_out) (act) when `norm` is given, or with `split` the row as two act numbers per entry [T, 2 width]
+    (see LoopInjection), or None: one launch in every case."""
+    T, D = x_in.shape
+    h = torch.empty((T, D), dtype=ctx.dtype, device=x_in.device) if norm is not None else None
+    s = torch.empty((T, 2 * D), dtype=ctx.dtype, device=x_in.device) if split else None
+    a = S.ResidualArgs(x_in=_p(x_in), base=_p(base), vec=_p(vec), y1=_p(y1), y2=_p(y2), x_out=_p(x_out), split=_p(s), w=_p(norm), b=_p(bias), h=_p(h),
+                       eps=eps, norm_kind=NORM_KINDS[kind], T=T, D=D, act_dtype=ctx.act)
+    S.check(S.lib().b2l_seq_residual_step(C.byref(a), ctx.stream), "b2l_seq_residual_step")
+    return s if split else h
+
+
+class LoopInjection:
+    """What stands before every pass of a looped stretch of layers:  x <- W_in [x; x0] + step[t],  x0 the embedding output and t
+    the number of the pass.
+
+    The half of the product on x0 is the same for every pass, so a portion computes it once (`start`).  The other half reads
+    the f32 stream: as it is (few tokens, float32 mode), or, where the library takes bf16 operands, as the pair hi + lo of
+    bf16 numbers in one product of twice the length, so that passing through W_in does not round the stream to 8 digits."""
+
+    def __init__(self, w_in: torch.Tensor, step: torch.Tensor) -> None:
+        D = w_in.shape[0]
+        if w_in.shape[1] != 2 * D or step.dim() != 2 or step.shape[1] != D:
+            raise ValueError(f"loop injection: {tuple(w_in.shape)} and {tuple(step.shape)} do not fit")
+        self.width, self.times = D, step.shape[0]
+        self.w_x, self.w_0 = w_in[:, :D].contiguous(), w_in[:, D:].contiguous()
+        self.w_xx = torch.cat([self.w_x, self.w_x], dim=1).contiguous() if w_in.dtype != torch.float32 else self.w_x
+        self.step = step.contiguous()
+
+    def wants_split(self, ctx: StepContext) -> bool:
+        """Whether `forward` takes the stream as the pair of act numbers that residual_step(split=True) returns."""
+        return ctx.T > FEW_TOKENS and ctx.dtype != torch.float32
+
+    def start(self, x0: torch.Tensor, h0: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        """W_in's half on the embedding output: x0 in f32, h0 the same in the activation type.  f32 [T, width]."""
+        if ctx.T > FEW_TOKENS:
+            return linear_f32(h0, self.w_0)
+        return self._few(self.w_0, x0, None, None, ctx)
+
+    def _few(self, w, x, base, vec, ctx: StepContext) -> torch.Tensor:
+        out = torch.empty((ctx.T, self.width), dtype=torch.float32, device=x.device)
+        S.check(S.lib().b2l_seq_linear_few(_p(w), _p(x), _p(base), _p(vec), _p(out), ctx.T, self.width, self.width, ctx.act, ctx.stream),
+                "b2l_seq_linear_few")
+        return out
+
+    def forward(self, x: torch.Tensor, split: Optional[torch.Tensor], base: torch.Tensor, t: int, ctx: StepContext, *, norm: torch.Tensor,
+                bias: Optional[torch.Tensor], kind: str, eps: float) -> Tuple[torch.Tensor, torch.Tensor]:
+        """The stream x (f32; `split` as residual_step returns it when `wants_split`) before pass t -> (new stream, its norm)."""
+        if ctx.T <= FEW_TOKENS:
+            new = self._few(self.w_x, x, base, self.step[t], ctx)
+            return new, norm_rows(new, norm, bias, kind, eps, ctx)
+        new = linear_f32(split, self.w_xx) if split is not None else F.linear(x, self.w_x)
+        return new, residual_step(new, new, ctx, base=base, vec=self.step[t], norm=norm, bias=bias, kind=kind, eps=eps)
 
 
 class DepthAverage:
@@ -721,8 +801,6 @@ class DepthAverage:
     output and X_(i+1) = x_i + (what layer i's sublayers add to their input x_i), the next layer's input is
     x_(i+1) = sum_(j <= i+1) avg_i[j] X_j (avg_i None: X_(i+1) itself, the ordinary residual stream).  `history` holds the
     X_j of one portion ([layers + 1, T, width] f32); `step` writes X_(i+1), forms x_(i+1) and the next norm in one launch."""
-
-    NORMS = {"rms": S.NORM_RMS, "layer": S.NORM_LAYER}
 
     def __init__(self, weights: List[Optional[torch.Tensor]]) -> None:
         self.avg = []
@@ -739,7 +817,7 @@ class DepthAverage:
         """Layer i's results y1 (+ y2) on its input x_in -> the next input in x_out (may be x_in), and its norm (act) when `norm` is given."""
         T, D = x_in.shape
         h = torch.empty((T, D), dtype=ctx.dtype, device=x_in.device) if norm is not None else None
-        S.check(S.lib().b2l_seq_depth_step(_p(y1), _p(y2), _p(x_in), _p(hist), i + 2, _p(self.avg[i]), _p(x_out), _p(norm), _p(bias), self.NORMS[kind],
+        S.check(S.lib().b2l_seq_depth_step(_p(y1), _p(y2), _p(x_in), _p(hist), i + 2, _p(self.avg[i]), _p(x_out), _p(norm), _p(bias), NORM_KINDS[kind],
                                            eps, _p(h), T, D, ctx.act, ctx.stream), "b2l_seq_depth_step")
         return h
 
@@ -808,10 +886,11 @@ class HyperConnection:
 class LatentAttention:
     """Causal softmax attention over a cached latent.
 
-        c_q = rmsnorm(W_dq h) w_q;  q = W_uq c_q, per head [dim unrotated | rot_dim rotated]
+        c_q = rmsnorm(W_dq h) w_q;  q = W_uq c_q, or (q_rank None) q = W_q h;  per head [dim unrotated | rot_dim rotated]
         [c' | k_r] = W_dkv h;  c = rmsnorm(c') w_kv (kv_rank);  k_r rotated by position, shared by all heads
         key_h = [W_uk,h c | k_r],  value_h = W_uv,h c,  score = q . key * scale
-        weights exp(s_j) / (exp(sink_h) + sum_j exp(s_j)),  y = W_o concat_h(sum_j weight_j value_j)
+        weights exp(s_j) / (exp(sink_h) + sum_j exp(s_j)),  y = W_o concat_h(sum_j weight_j value_j), with `gate` times
+        sigmoid(W_g h) per channel before W_o
 
     over every earlier position, or with `window` over the query's own position and the window - 1 before it; without a
     `sink` tensor the softmax is the ordinary one.  A YaRN `scaling` of the rotation stretches the slow frequencies and
@@ -819,7 +898,8 @@ class LatentAttention:
 
     Only [c | k_r] is cached per position.  Single tokens and short portions attend in the latent space: the query is
     multiplied by W_uk once (q' = W_uk,h^T q_h), scores are q' . c + q_r . k_r, the weighted sum of latents is mapped
-    through W_uv afterwards; every head reads the same cached row, once.  Portions of `expand_from` tokens or more
+    through W_uv afterwards (up to FEW_TOKENS tokens in the launch that merges the key splits and gates, and with direct
+    queries W_uk is applied in the launch that turns the rotated parts); every head reads the same cached row, once.  Portions of `expand_from` tokens or more
     expand [value_h | key_h] of every cached position with one product and attend per head, which costs several times
     fewer operations per (query, key) pair.  Both forms run the same kernel.  `rot`: {"base", "dims"} on the first
     `dims` entries of the rotated part, pairs (2i, 2i+1) when `interleaved`."""
@@ -827,9 +907,9 @@ class LatentAttention:
     expand_from: int = 64                 # portions at least this long take the expanded form
     expand_limit: int = 1 << 31           # ... unless the expansion would have more elements than this
 
-    def __init__(self, name: str, W: Dict[str, torch.Tensor], p: str, *, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: int,
+    def __init__(self, name: str, W: Dict[str, torch.Tensor], p: str, *, heads: int, dim: int, rot_dim: int, vdim: int, q_rank: Optional[int],
                  kv_rank: int, scale: float, eps: float, rot: Optional[dict], max_positions: int, interleaved: bool = True,
-                 window: Optional[int] = None) -> None:
+                 window: Optional[int] = None, gate: bool = False) -> None:
         if max_positions <= 0:
             raise ValueError("latent attention caches every position: it needs max_positions")
         self.window = int(window) if window else 0
@@ -837,14 +917,20 @@ class LatentAttention:
             raise ValueError("latent attention: negative window")
         self.name, self.H, self.dn, self.dr, self.dv, self.rq, self.rk = name, heads, dim, rot_dim, vdim, q_rank, kv_rank
         self.scale, self.eps, self.max_positions, self.interleaved = float(scale), eps, int(max_positions), bool(interleaved)
-        self.w_in, (self.o_q, self.o_kv) = stack_rows([W[p + "dq"], W[p + "dkv"]])
-        assert W[p + "dq"].shape[0] == q_rank and W[p + "dkv"].shape[0] == kv_rank + rot_dim, "latent attention: down-projections do not fit"
-        self.q_norm, self.kv_norm = W[p + "dq.norm"].contiguous(), W[p + "dkv.norm"].contiguous()
-        self.w_uq = W[p + "uq"].contiguous()
-        assert self.w_uq.shape == (heads * (dim + rot_dim), q_rank), "latent attention: query up-projection does not fit"
+        w_q = W[p + "q"] if q_rank is None else W[p + "dq"]
+        assert w_q.shape[0] == (heads * (dim + rot_dim) if q_rank is None else q_rank) and W[p + "dkv"].shape[0] == kv_rank + rot_dim, \
+            "latent attention: the input projections do not fit"
+        self.w_in, offs = stack_rows([w_q, W[p + "dkv"]] + ([W[p + "g"]] if gate else []))
+        self.o_q, self.o_kv, self.o_g = offs[0], offs[1], (offs[2] if gate else None)
+        assert not gate or W[p + "g"].shape[0] == heads * vdim, "latent attention: the gate does not fit"
+        self.kv_norm = W[p + "dkv.norm"].contiguous()
+        self.q_norm = self.w_uq = None
+        if q_rank is not None:
+            self.q_norm, self.w_uq = W[p + "dq.norm"].contiguous(), W[p + "uq"].contiguous()
+            assert self.w_uq.shape == (heads * (dim + rot_dim), q_rank), "latent attention: query up-projection does not fit"
         uk, uv = W[p + "uk"].reshape(heads, dim, kv_rank), W[p + "uv"].reshape(heads, vdim, kv_rank)
         self.w_uk = uk.contiguous()                                                            # q' = q_h W_uk,h
-        self.w_uv_t = uv.transpose(1, 2).contiguous()                                          # value = o' W_uv,h^T
+        self.w_uv = uv.contiguous()                                                            # value = W_uv,h o'
         self.w_expand = torch.cat([uv, uk], dim=1).reshape(heads * (vdim + dim), kv_rank).contiguous()   # per head [value | key] rows
         self.sink = W[p + "sink"].to(torch.float32).contiguous() if (p + "sink") in W else None
         self.w_o = W[p + "o"].contiguous()
@@ -871,50 +957,87 @@ class LatentAttention:
             return 1
         return max(1, min(-(-444 // ctas), -(-n_keys // 32)))
 
-    def _attend(self, ctx: StepContext, out: torch.Tensor, vdim: int, splits: int, **kw) -> None:
-        work = torch.empty((splits, ctx.T * self.H, vdim + 2), dtype=torch.float32, device=out.device) if splits > 1 else None
+    def _attend(self, ctx: StepContext, out: Optional[torch.Tensor], vdim: int, splits: int, **kw) -> Optional[torch.Tensor]:
+        """The attention kernel into `out`, or (out None) its partial results: f32 [splits, T * heads, vdim + 2]."""
+        dev = ctx.meta.device
+        work = torch.empty((splits, ctx.T * self.H, vdim + 2), dtype=torch.float32, device=dev) if splits > 1 or out is None else None
         a = S.LatentAttnArgs(sink=_p(self.sink), meta=_p(ctx.meta), out=_p(out), ldo=self.H * vdim, work=_p(work), scale=self.scale, T=ctx.T,
-                             heads=self.H, vdim=vdim, splits=splits, act_dtype=ctx.act, window=self.window, **kw)
+                             heads=self.H, vdim=vdim, splits=splits, act_dtype=ctx.act, window=self.window, partial=int(out is None), **kw)
         S.check(S.lib().b2l_seq_latent_attention(C.byref(a), ctx.stream), "b2l_seq_latent_attention")
+        return work
+
+    def _rope(self, x: torch.Tensor, off: int, rot_off: int, size: int, out: torch.Tensor, ctx: StepContext) -> None:
+        """Entries [off, off + size) of every head of x -> out (f32), the rotated entries from rot_off on turned by position."""
+        H, dq = self.H, self.dn + self.dr
+        S.check(S.lib().b2l_seq_rope(_p(x, off), H * dq, int(x.dtype == torch.float32), _p(self.freq), self.rot_dims, int(self.interleaved), rot_off, 1.0,
+                                     self.rot_mult, _p(ctx.meta), _p(out), H * size, 1, ctx.T, H, size, dq, size, ctx.act, ctx.stream), "b2l_seq_rope")
+
+    def _queries(self, h: torch.Tensor, cache: torch.Tensor, ctx: StepContext, expanded: bool):
+        """Projections of the portion: appends its latents to the cache and returns (gate, q32, q_lat, q_rot): q32 f32
+        [T, H * (dim + rot_dim)] for the expanded form, or q_lat f32 [H, T, rank] and q_rot f32 [T, H, rot_dim]."""
+        lib, T, dev, H, dn, dr = S.lib(), ctx.T, h.device, self.H, self.dn, self.dr
+        dq, f32 = dn + dr, h.dtype == torch.float32
+        proj = linear_f32(h, self.w_in)
+        gate = (proj, self.o_g) if self.o_g is not None else None
+        q32 = torch.empty((T, H * dq), dtype=torch.float32, device=dev) if expanded else None
+        q_rot = torch.empty((T, H, max(dr, 1)), dtype=torch.float32, device=dev) if not expanded else None
+        qn = q_lat = None
+        if self.rq is None:
+            if not expanded:
+                if T <= FEW_TOKENS:
+                    q_lat = torch.empty((H, T, self.rk), dtype=torch.float32, device=dev)
+                else:
+                    qn = torch.empty((H, T, dn), dtype=h.dtype, device=dev)
+            a = S.LatentOperandsArgs(proj=_p(proj), ld=proj.shape[1], q_off=self.o_q, kv_off=self.o_kv, heads=H, dn=dn, dr=dr, rank=self.rk, w_kv=_p(self.kv_norm),
+                                     freq=_p(self.freq), rot_dims=self.rot_dims, interleaved=int(self.interleaved), rot_mult=self.rot_mult, eps=self.eps,
+                                     meta=_p(ctx.meta), cache=_p(cache), max_pos=self.max_positions, q_full=_p(q32), q_nope=_p(qn), q_rot=_p(q_rot),
+                                     w_uk=_p(self.w_uk) if q_lat is not None else None, q_lat=_p(q_lat), T=T, act_dtype=ctx.act)
+            S.check(lib.b2l_seq_latent_operands(C.byref(a), ctx.stream), "b2l_seq_latent_operands")
+        else:
+            cq = torch.empty((T, self.rq), dtype=h.dtype, device=dev)
+            S.check(lib.b2l_seq_latent_prep(_p(proj), proj.shape[1], self.o_q, self.rq, _p(self.q_norm), _p(cq), self.o_kv, self.rk, _p(self.kv_norm),
+                                            dr, _p(self.freq), self.rot_dims, int(self.interleaved), self.rot_mult, self.eps, _p(ctx.meta), _p(cache),
+                                            self.max_positions, T, ctx.act, ctx.stream), "b2l_seq_latent_prep")
+            q = linear(cq, self.w_uq)                                               # [T, H * (dim + rot_dim)]
+            if expanded:
+                self._rope(q, 0, dn, dq, q32, ctx)
+            else:
+                qn = q.view(T, H, dq)[:, :, :dn].transpose(0, 1)                     # [H, T, dim]
+                if dr:
+                    self._rope(q, dn, 0, dr, q_rot, ctx)
+        if not expanded and q_lat is None:
+            q_lat = torch.bmm(qn, self.w_uk) if f32 else torch.bmm(qn, self.w_uk, out_dtype=torch.float32)
+        return gate, q32, q_lat, q_rot
 
     def forward(self, h: torch.Tensor, ctx: StepContext) -> torch.Tensor:
-        lib, T, dev, H = S.lib(), ctx.T, h.device, self.H
-        proj = linear_f32(h, self.w_in)
-        cq = torch.empty((T, self.rq), dtype=h.dtype, device=dev)
-        cache = ctx.state[self.name + ".kv"]
-        Kd = self.rk + self.dr
-        S.check(lib.b2l_seq_latent_prep(_p(proj), proj.shape[1], self.o_q, self.rq, _p(self.q_norm), _p(cq), self.o_kv, self.rk, _p(self.kv_norm),
-                                        self.dr, _p(self.freq), self.rot_dims, int(self.interleaved), self.rot_mult, self.eps, _p(ctx.meta), _p(cache),
-                                        self.max_positions, T, ctx.act, ctx.stream), "b2l_seq_latent_prep")
-        dq, f32 = self.dn + self.dr, h.dtype == torch.float32
-        q = linear(cq, self.w_uq)                                                   # [T, H * (dim + rot_dim)]
-        shared_b = dict(key_b=_p(cache, self.rk), ldkb=Kd, slot_stride_b=self.max_positions * Kd, n_b=self.dr)
+        lib, T, dev, H, dn, dv, dr = S.lib(), ctx.T, h.device, self.H, self.dn, self.dv, self.dr
+        cache, Kd, dq = ctx.state[self.name + ".kv"], self.rk + self.dr, self.dn + self.dr
         n_pos = None if ctx.pos_hint is None or ctx.slot_hint is None else ctx.pos_hint + T
-        if n_pos is not None and T >= self.expand_from and n_pos * H * (self.dv + self.dn) <= self.expand_limit:
-            # expanded form: [value_h | key_h] of positions 0 .. n_pos-1 from the cached latents, one product
-            q32 = torch.empty((T, H * dq), dtype=torch.float32, device=dev)
-            S.check(lib.b2l_seq_rope(_p(q), H * dq, int(f32), _p(self.freq), self.rot_dims, int(self.interleaved), self.dn, 1.0, self.rot_mult, _p(ctx.meta),
-                                     _p(q32), H * dq, 1, T, H, dq, dq, dq, ctx.act, ctx.stream), "b2l_seq_rope")
+        expanded = n_pos is not None and T >= self.expand_from and n_pos * H * (dv + dn) <= self.expand_limit
+        gate, q32, q_lat, q_rot = self._queries(h, cache, ctx, expanded)
+        gp, ldg = (_p(*gate), gate[0].shape[1]) if gate is not None else (None, 0)
+        shared_b = dict(key_b=_p(cache, self.rk), ldkb=Kd, slot_stride_b=self.max_positions * Kd, n_b=dr)
+        att = torch.empty((T, H * dv), dtype=h.dtype, device=dev)
+        if expanded:                            # [value_h | key_h] of positions 0 .. n_pos-1 from the cached latents, one product
             lo = max(0, ctx.pos_hint - self.window + 1) if self.window else 0       # the first position any query of the portion sees
             kv = linear(cache[ctx.slot_hint, lo:n_pos, :self.rk], self.w_expand)     # [n_pos - lo, H * (vdim + dim)]: row j - lo is position j
-            att = torch.empty((T, H * self.dv), dtype=h.dtype, device=dev)
-            self._attend(ctx, att, self.dv, self._splits(ctx, 1), q_a=_p(q32), ldqa_t=H * dq, ldqa_h=dq, q_b=_p(q32, self.dn), ldqb_t=H * dq,
-                         ldqb_h=dq, key_a=_p(kv, -lo * H * (self.dv + self.dn)), ldka=H * (self.dv + self.dn), hska=self.dv + self.dn, slot_stride_a=0, n_a=self.dv + self.dn,
-                         score_off=self.dv, heads_per_group=1, **shared_b)
+            self._attend(ctx, att, dv, self._splits(ctx, 1), q_a=_p(q32), ldqa_t=H * dq, ldqa_h=dq, q_b=_p(q32, dn), ldqb_t=H * dq, ldqb_h=dq,
+                         key_a=_p(kv, -lo * H * (dv + dn)), ldka=H * (dv + dn), hska=dv + dn, slot_stride_a=0, n_a=dv + dn, score_off=dv, heads_per_group=1,
+                         gate=gp, ldg=ldg, **shared_b)
             return linear(att, self.w_o)
-        # latent form
-        qn = q.view(T, H, dq)[:, :, :self.dn].transpose(0, 1)                        # [H, T, dim]
-        q_lat = torch.bmm(qn, self.w_uk) if f32 else torch.bmm(qn, self.w_uk, out_dtype=torch.float32)     # [H, T, rank] f32
-        q_rot = torch.empty((T, H, max(self.dr, 1)), dtype=torch.float32, device=dev)
-        if self.dr:
-            S.check(lib.b2l_seq_rope(_p(q, self.dn), H * dq, int(f32), _p(self.freq), self.rot_dims, int(self.interleaved), 0, 1.0, self.rot_mult, _p(ctx.meta),
-                                     _p(q_rot), H * self.dr, 1, T, H, self.dr, dq, self.dr, ctx.act, ctx.stream), "b2l_seq_rope")
+        latent = dict(q_a=_p(q_lat), ldqa_t=self.rk, ldqa_h=T * self.rk, q_b=_p(q_rot), ldqb_t=H * max(dr, 1), ldqb_h=max(dr, 1), key_a=_p(cache), ldka=Kd, hska=0,
+                      slot_stride_a=self.max_positions * Kd, n_a=self.rk, score_off=0, heads_per_group=H, **shared_b)
+        splits = self._splits(ctx, H)
+        if T <= FEW_TOKENS:                     # merge of the splits, W_uv and gate in one launch
+            work = self._attend(ctx, None, self.rk, splits, **latent)
+            S.check(lib.b2l_seq_latent_up(_p(work), _p(self.sink), _p(self.w_uv), gp, ldg, _p(att), H * dv, T, H, self.rk, dv, splits, ctx.act, ctx.stream),
+                    "b2l_seq_latent_up")
+            return linear(att, self.w_o)
         o_lat = torch.empty((T, H * self.rk), dtype=h.dtype, device=dev)
-        self._attend(ctx, o_lat, self.rk, self._splits(ctx, H), q_a=_p(q_lat), ldqa_t=self.rk, ldqa_h=T * self.rk, q_b=_p(q_rot),
-                     ldqb_t=H * max(self.dr, 1), ldqb_h=max(self.dr, 1), key_a=_p(cache), ldka=Kd, hska=0, slot_stride_a=self.max_positions * Kd,
-                     n_a=self.rk, score_off=0, heads_per_group=H, **shared_b)
-        v = torch.bmm(o_lat.view(T, H, self.rk).transpose(0, 1), self.w_uv_t)        # [H, T, vdim]
-        return linear(v.transpose(0, 1).reshape(T, H * self.dv), self.w_o)
+        self._attend(ctx, o_lat, self.rk, splits, **latent)
+        v = torch.bmm(o_lat.view(T, H, self.rk).transpose(0, 1), self.w_uv.transpose(1, 2))      # [H, T, vdim]
+        S.check(lib.b2l_seq_head_gate(_p(v), dv, T * dv, gp, ldg, _p(att), H * dv, T, H, dv, ctx.act, ctx.stream), "b2l_seq_head_gate")
+        return linear(att, self.w_o)
 
 
 # ------------------------------------------------------------------------------------------------ retention
@@ -974,23 +1097,25 @@ class MoEFeedForward:
         (steers the choice only); experts form `groups` equal groups of neighbours; a group is worth the sum of its
         `group_top` largest choice scores (1: its best); only experts of the `keep` best groups can be chosen; the `top`
         largest choice scores win;  weight = s / (sum of the chosen s + 1e-20) when `renormalize`, else s itself, times
-        `weight_scale`
+        `weight_scale`;  or (`score` = "chosen_softmax") the choice is made on the logits z = W_router h + bias and the weights
+        are the softmax of z over the chosen experts
         expert e < experts: W_down unit(W_gate x, W_up x) with unit(a, b) = act(a) * b, or the clamped unit
         min(a, limit) * sigmoid(1.702 min(a, limit)) * (clamp(b, -limit, limit) + 1) (`act` = "clamped_swish");
         x = h and the weight scales the expert's output, or (`weight_on` = "input") x = weight * h and the outputs are
         summed unweighted;  the last `identity` outputs of the router: h itself
+        with `shared_ff` one more expert of that size runs on every token's h and is added unweighted
 
     A few tokens (also the captured single-token step) run with the expert index read on the device; longer portions
     sort the assignments by expert and run one pair of products per expert that received tokens."""
 
-    SMALL = 4
+    SMALL = FEW_TOKENS
     grouped = True        # bf16, 16-byte rows: the library's grouped product instead of one product per expert
 
-    SCORES = {"softmax": S.SCORE_SOFTMAX, "sigmoid": S.SCORE_SIGMOID}
+    SCORES = {"softmax": S.SCORE_SOFTMAX, "sigmoid": S.SCORE_SIGMOID, "chosen_softmax": S.SCORE_CHOSEN_SOFTMAX}
 
     def __init__(self, W: Dict[str, torch.Tensor], p: str, *, experts: int, identity: int, top: int, groups: int, keep: int, ff: int,
                  act: str = "silu", limit: float = 0.0, score: str = "softmax", renormalize: bool = True, weight_on: str = "output",
-                 group_top: int = 1, weight_scale: float = 1.0) -> None:
+                 group_top: int = 1, weight_scale: float = 1.0, shared_ff: int = 0) -> None:
         self.group_top, self.weight_scale = int(group_top), float(weight_scale)
         if self.group_top < 1:
             raise ValueError("routed experts: a group's score needs at least its best member")
@@ -1004,11 +1129,14 @@ class MoEFeedForward:
         if score not in self.SCORES or weight_on not in ("output", "input"):
             raise ValueError(f"routed experts: unknown score function {score!r} or weight placement {weight_on!r}")
         self.score, self.renorm, self.weight_input = self.SCORES[score], int(bool(renormalize)), int(weight_on == "input")
+        if score == "chosen_softmax" and not renormalize:
+            raise ValueError("routed experts: a softmax over the chosen logits sums to one")
         if self.weight_input and self.I:
             raise ValueError("routed experts: identity experts with weights on the input are not built")
         self.w_router = W[p + "router"].contiguous()
         assert self.w_router.shape[0] == self.n, "routed experts: the router does not have experts + identity outputs"
-        self.correction = W[p + "correction"].to(torch.float32).contiguous() if (p + "correction") in W else None
+        bias = p + ("router.b" if score == "chosen_softmax" else "correction")      # the kernels' `correction`: of the choice, or of the logits
+        self.correction = W[bias].to(torch.float32).contiguous() if bias in W else None
         dev, dt = self.w_router.device, W[p + "router"].dtype
         if self.E:
             self.w_gu = torch.stack([torch.cat([W[f"{p}e{e}.gate"], W[f"{p}e{e}.up"]], dim=0) for e in range(self.E)]).contiguous()
@@ -1016,6 +1144,10 @@ class MoEFeedForward:
             assert self.w_gu.shape[1] == 2 * self.ff, "routed experts: expert size does not fit"
         else:
             self.w_gu = self.w_down = torch.zeros(0, dtype=dt, device=dev)
+        self.shared: Optional[GatedMLP] = None
+        if shared_ff:
+            self.shared = GatedMLP(W[p + "shared.gate"], W[p + "shared.up"], W[p + "shared.down"], act=act, limit=limit)
+            assert self.shared.ff == int(shared_ff), "routed experts: the shared expert does not have its size"
         self.last_idx: Optional[torch.Tensor] = None       # the routing of the last call (tests, diagnostics)
 
     def state_specs(self) -> Dict[str, StateSpec]:
@@ -1046,11 +1178,14 @@ class MoEFeedForward:
         y = torch.empty((T, D), dtype=h.dtype, device=dev)
         N = T * top
         if T <= self.SMALL or E == 0:
-            mid = torch.empty((N, ff), dtype=h.dtype, device=dev)
+            sh = self.shared
+            mid = torch.empty((N * ff + (T * sh.ff if sh is not None else 0),), dtype=h.dtype, device=dev)
             S.check(lib.b2l_seq_moe_experts_small(_p(h), D, _p(self.w_gu) if E else None, _p(self.w_down) if E else None, _p(idx), _p(wgt), _p(mid),
-                                                  _p(y), D, T, D, ff, E, top, self.act, self.limit, self.weight_input, ctx.act, ctx.stream),
+                                                  _p(y), D, T, D, ff, E, top, self.act, self.limit, self.weight_input, _p(sh.w_in) if sh is not None else None,
+                                                  _p(sh.w_down) if sh is not None else None, sh.ff if sh is not None else 0, ctx.act, ctx.stream),
                     "b2l_seq_moe_experts_small")
             return y
+        y_shared = self.shared.forward(h, ctx) if self.shared is not None else None
         meta = torch.empty((2 * (E + 1) + 2 * N,), dtype=torch.int32, device=dev)
         offsets, cursor, perm, inv = meta[:E + 1], meta[E + 1:2 * E + 2], meta[2 * E + 2:2 * E + 2 + N], meta[2 * E + 2 + N:]
         S.check(lib.b2l_seq_moe_sort(_p(idx), N, E, _p(offsets), _p(cursor), _p(perm), _p(inv), ctx.stream), "b2l_seq_moe_sort")
@@ -1075,6 +1210,6 @@ class MoEFeedForward:
             for e in range(E):
                 if off[e + 1] > off[e]:
                     torch.mm(mid[off[e]:off[e + 1]], self.w_down[e].t(), out=yg[off[e]:off[e + 1]])
-        S.check(lib.b2l_seq_moe_combine(_p(yg), _p(inv), None if self.weight_input else _p(wgt), _p(h), D, _p(y), D, T, D, top, ctx.act,
-                                        ctx.stream), "b2l_seq_moe_combine")
+        S.check(lib.b2l_seq_moe_combine(_p(yg), _p(inv), None if self.weight_input else _p(wgt), _p(h), D, _p(y_shared), D, _p(y), D, T, D, top,
+                                        ctx.act, ctx.stream), "b2l_seq_moe_combine")
         return y

@@ -56,6 +56,13 @@ def _load_lukupel(model_dir: str, dtype: torch.dtype, device: torch.device, max_
     return lukupel.load(model_dir, dtype=dtype, device=device, max_positions=max_positions)
 
 
+@register("Malulorn")
+def _load_malulorn(model_dir: str, dtype: torch.dtype, device: torch.device, max_positions: int, config: dict):
+    from . import malulorn
+
+    return malulorn.load(model_dir, dtype=dtype, device=device, max_positions=max_positions)
+
+
 @register("LLaMA")
 def _load_llama(model_dir: str, dtype: torch.dtype, device: torch.device, max_positions: int, config: dict):
     """config.json: {"architecture": "LLaMA", "name": "7B" | sizes..., "quantize": null | "gptq.int4" | ..., "checkpoint": file}."""

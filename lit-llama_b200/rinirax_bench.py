@@ -179,7 +179,7 @@ def kernel_table(model, engine, T: int, device, timer, peaks: dict) -> List[dict
             add(f"{name}, {form} form)", tt, t, nbl, fl, f"f32 scores on CUDA cores, {kq:.0f} keys per query, {splits} key split(s)")
         lat.window, lat.sink = Wn, None
         t = timer(lambda: lat.forward(hh, ctx))
-        wb = (lat.w_in.numel() + lat.w_uq.numel() + lat.w_uk.numel() + lat.w_uv_t.numel() + lat.w_o.numel()) * es
+        wb = (lat.w_in.numel() + lat.w_uq.numel() + lat.w_uk.numel() + lat.w_uv.numel() + lat.w_o.numel()) * es
         add("LatentAttention whole (5 products + prep + rotation + attention)", tt, t, wb + 2 * tt * D * es)
         # ---- the recurrence: a state per channel against a matrix state per head
         n = gru.width

@@ -126,7 +126,7 @@ def kernel_table(model, engine, T: int, device, timer, peaks: dict) -> List[dict
             "seq_block_attention_tile_kernel" if tt > 1 else "seq_block_attention_kernel", tt, t, nb, fl,
             f"f32 scores on CUDA cores, {splits} key split(s)")
         t = timer(lambda: att.forward(hh, ctx))
-        wb = (att.w_in.numel() + att.w_uq.numel() + att.w_uk.numel() + att.w_uv_t.numel() + att.w_o.numel()) * es
+        wb = (att.w_in.numel() + att.w_uq.numel() + att.w_uk.numel() + att.w_uv.numel() + att.w_o.numel()) * es
         add("LatentAttention whole (5 products + prep + rotation + attention)", "attention branch", tt, t, wb + nb, fl + 2.0 * tt * wb / es)
         t = timer(lambda: ret.forward(hh, ctx))
         st = ret.H * ret.K * ret.V * 4 * 2
