@@ -100,8 +100,8 @@ __global__ void __launch_bounds__(128) seq_latent_prep_kernel(const float* __res
 // Every CTA computes the angles it needs once per pair.
 constexpr int LAT_ABS_COLS = 128;
 
-template <typename act_t>
-__global__ void __launch_bounds__(256) seq_latent_operands_kernel(b2l_seq_latent_operands_args a, int chunks) {
+template <typename act_t, bool ABSORB>
+__global__ void __launch_bounds__(256) seq_latent_operands_kernel(b2l_seq_latent_operands_args a, int chunks, int quads) {
   extern __shared__ __align__(16) float op_smem[];                // cos | sin per pair, then (absorbed) q [dn]
   __shared__ float red[32];
   __shared__ float part[4][LAT_ABS_COLS];
@@ -111,7 +111,7 @@ __global__ void __launch_bounds__(256) seq_latent_operands_kernel(b2l_seq_latent
   float* cs = op_smem;
   float* sn = cs + half;
   const int b = (int)blockIdx.y - 1;
-  const int h0 = a.q_lat ? b / chunks : 0, chunk = a.q_lat ? b - h0 * chunks : 0;
+  const int h0 = ABSORB ? b / chunks : 0, chunk = ABSORB ? b - h0 * chunks : 0;
   if (b < 0 || chunk == 0) {
     for (int i = tid; i < half; i += blockDim.x) {
       float s, c;
@@ -141,32 +141,50 @@ __global__ void __launch_bounds__(256) seq_latent_operands_kernel(b2l_seq_latent
   }
   const float* q = row + a.q_off;
   float* sq = sn + half;
-  if (a.q_lat)
+  if (ABSORB)
     for (int i = tid; i < a.dn; i += blockDim.x) sq[i] = q[(size_t)h0 * dq + i];
   __syncthreads();
-  // rotated parts of the heads [h0, h1)
+  if (!ABSORB && quads) {                                         // q_full, interleaved, everything in groups of four: copy and turn
+    float* o = a.q_full + (size_t)t * a.heads * dq;
+    for (int i = tid * 4; i < a.heads * dq; i += blockDim.x * 4) {
+      float4 v = *reinterpret_cast<const float4*>(q + i);
+      const int j = i % dq - a.dn;
+      if (j >= 0 && j < a.rot_dims) {
+        const int p0 = j >> 1;
+        v = make_float4(v.x * cs[p0] - v.y * sn[p0], v.y * cs[p0] + v.x * sn[p0], v.z * cs[p0 + 1] - v.w * sn[p0 + 1], v.w * cs[p0 + 1] + v.z * sn[p0 + 1]);
+      }
+      *reinterpret_cast<float4*>(o + i) = v;
+    }
+    return;
+  }
+  const int warp = tid >> 5, lane = tid & 31, nw = blockDim.x >> 5;
+  // rotated parts: a warp per head (absorbed: of the CTA's own head, by its first warp)
   if (chunk == 0) {
-    const int h1 = a.q_lat ? h0 + 1 : a.heads, rest = a.dr - a.rot_dims, per = half + rest;
-    for (int i = tid; i < (h1 - h0) * per; i += blockDim.x) {
-      const int hd = h0 + i / per, j = i % per;
+    const int h1 = ABSORB ? h0 + 1 : a.heads;
+    for (int hd = h0 + warp; hd < h1; hd += nw) {
       const float* p = q + (size_t)hd * dq + a.dn;
       float* o = a.q_full ? a.q_full + ((size_t)t * a.heads + hd) * dq + a.dn : a.q_rot + ((size_t)t * a.heads + hd) * a.dr;
-      if (j < half) {
+      for (int j = lane; j < half; j += 32) {
         const int iu = a.interleaved ? 2 * j : j, iv = a.interleaved ? 2 * j + 1 : j + half;
         const float u = p[iu], v = p[iv];
         o[iu] = u * cs[j] - v * sn[j];
         o[iv] = v * cs[j] + u * sn[j];
-      } else {
-        o[a.rot_dims + j - half] = p[a.rot_dims + j - half];
       }
+      for (int j = a.rot_dims + lane; j < a.dr; j += 32) o[j] = p[j];
     }
   }
-  if (a.q_lat == nullptr) {
-    for (int i = tid; i < a.heads * a.dn; i += blockDim.x) {
-      const int hd = i / a.dn, j = i - hd * a.dn;
-      const float v = q[(size_t)hd * dq + j];
-      if (a.q_full) a.q_full[((size_t)t * a.heads + hd) * dq + j] = v;
-      else st_act((act_t*)a.q_nope, ((size_t)hd * a.T + t) * a.dn + j, v);
+  if (!ABSORB) {
+    for (int hd = warp; hd < a.heads; hd += nw) {
+      const float* p = q + (size_t)hd * dq;
+      if (a.q_full) {
+        float* o = a.q_full + ((size_t)t * a.heads + hd) * dq;
+#pragma unroll 4
+        for (int j = lane; j < a.dn; j += 32) o[j] = p[j];
+      } else {
+        act_t* o = (act_t*)a.q_nope + ((size_t)hd * a.T + t) * a.dn;
+#pragma unroll 4
+        for (int j = lane; j < a.dn; j += 32) st_act(o, j, p[j]);
+      }
     }
     return;
   }
@@ -218,7 +236,7 @@ __global__ void __launch_bounds__(LAT_THREADS, VI <= 4 ? 3 : 1) seq_latent_atten
   extern __shared__ __align__(16) float lat_smem[];
   const int Kall = a.n_a + a.n_b, Kp = (Kall + 3) & ~3;
   const int s0 = a.score_off & ~3, Qp = Kp - s0;                       // scores run over d in [s0, Kp), q is zero below score_off
-  const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int hpg = a.heads_per_group, group = blockIdx.z;
   const int rows_cta = row_warps * LAT_RW, R = a.T * hpg;
   float* kT = lat_smem;
@@ -605,7 +623,13 @@ extern "C" int b2l_seq_latent_operands(const b2l_seq_latent_operands_args* a, b2
   const size_t smem = sizeof(float) * ((size_t)a->rot_dims + a->dn);
   B2L_CHECK_SUPPORTED(gy <= 65535 && smem <= 40 * 1024, "b2l_seq_latent_operands: %d heads of %d + %d entries over a latent of %d are too many", a->heads, a->dn,
                       a->dr, a->rank);
-  B2L_SEQ_DISPATCH(a->act_dtype, (seq_latent_operands_kernel<act_t><<<dim3(a->T, (unsigned)gy), 256, smem, (cudaStream_t)stream>>>(*a, chunks)));
+  const int quads = a->q_full && a->interleaved && a->dn % 4 == 0 && a->dr % 4 == 0 && a->rot_dims % 4 == 0 && a->q_off % 4 == 0 && a->ld % 4 == 0 &&
+                    al16(a->proj) && al16(a->q_full);
+  const dim3 grid(a->T, (unsigned)gy);
+  B2L_SEQ_DISPATCH(a->act_dtype, {
+    if (a->q_lat) seq_latent_operands_kernel<act_t, true><<<grid, 256, smem, (cudaStream_t)stream>>>(*a, chunks, 0);
+    else seq_latent_operands_kernel<act_t, false><<<grid, 256, smem, (cudaStream_t)stream>>>(*a, chunks, quads);
+  });
   B2L_LAUNCH_CHECK("seq_latent_operands_kernel");
   return 0;
 }

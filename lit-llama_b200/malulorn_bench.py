@@ -61,18 +61,23 @@ def kernel_table(model, engine, T: int, device, timer, peaks: dict) -> List[dict
         w, b, h = torch.ones(D, dtype=dt, device=device), torch.zeros(D, dtype=dt, device=device), torch.empty(tt, D, dtype=dt, device=device)
         # ---- residual step
         nb = tt * D * (es + 4 + 4 + es)
-        add("seq_residual_step_kernel (sum, layer norm)", tt, timer(lambda: M.residual_step(x, x, ctx, y1=y, norm=w, bias=b, kind="layer", eps=eps)), nb)
+
+        def residual(**kw):
+            a = S.ResidualArgs(x_in=p(x), x_out=p(x), eps=eps, norm_kind=S.NORM_LAYER, T=tt, D=D, act_dtype=act, **kw)
+            return timer(lambda: S.check(lib.b2l_seq_residual_step(C.byref(a), st), "k"))
+
+        add("seq_residual_step_kernel (sum, layer norm)", tt, residual(y1=p(y), w=p(w), b=p(b), h=p(h)), nb)
         t = timer(lambda: S.check(lib.b2l_seq_depth_step(p(y), None, p(x), p(x2), 1, None, p(x), p(w), p(b), S.NORM_LAYER, eps, p(h), tt, D, act, st), "k"))
         add("  like: seq_depth_step_kernel (sum, history entry, layer norm)", tt, t, nb + tt * D * 4)
         # ---- injection before a pass
         inj = model.inject
         base = inj.start(x, hh, ctx)
         if tt > M.FEW_TOKENS:
-            add("seq_residual_step_kernel (sum, split pair)", tt, timer(lambda: M.residual_step(x, x, ctx, y1=y, split=True)), tt * D * (es + 4 + 4 + 2 * es))
+            pair = torch.empty(tt, 2 * D, dtype=dt, device=device)
+            add("seq_residual_step_kernel (sum, split pair)", tt, residual(y1=p(y), split=p(pair)), tt * D * (es + 4 + 4 + 2 * es))
             add("seq_residual_step_kernel (product + base + step vector, layer norm)", tt,
-                timer(lambda: M.residual_step(x, x, ctx, base=base, vec=inj.step[0], norm=w, bias=b, kind="layer", eps=eps)), tt * D * (4 + 4 + 4 + es))
-            sp = M.residual_step(x, None, ctx, split=True)
-            t = timer(lambda: inj.forward(x, sp, base, 0, ctx, norm=w, bias=b, kind="layer", eps=eps))
+                residual(base=p(base), vec=p(inj.step[0]), w=p(w), b=p(b), h=p(h)), tt * D * (4 + 4 + 4 + es))
+            t = timer(lambda: inj.forward(x, pair, base, 0, ctx, norm=w, bias=b, kind="layer", eps=eps))
             add("LoopInjection whole (product of the pair + step)", tt, t, 2 * D * D * es + tt * D * (2 * es + 4 * 4 + es), 4.0 * tt * D * D)
         else:
             new = torch.empty(tt, D, device=device)
