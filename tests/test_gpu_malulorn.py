@@ -431,7 +431,7 @@ def test_attention_denominator_takes_its_share():
                 assert torch.allclose(got[t], want, rtol=1e-4, atol=1e-6), (level, sizes, t)
 
 
-@pytest.mark.parametrize("coef,every", [(0.3, 128), (0.5, 1), (-0.2, 3), (0.1, 1000), (0.0, 7)])
+@pytest.mark.parametrize("coef,every", [(0.35, 96), (0.5, 1), (-0.2, 3), (0.1, 1000), (0.0, 7)])
 def test_query_temperature_steps_at_its_positions(coef, every):
     P, S, M = _pkg()
     H, G, K, T = 3, 1, 10, 9
